@@ -4,7 +4,7 @@ Layers whose mixers ask for the same ``KVCacheSpec`` form a group.  A group
 has its own page pool (one tensor per layer, the same page id naming the same
 page in each of the group's layers, as the reference's single id does across
 all layers, rosellm/roseinfer/engine.py:4370-4408), its own allocator and its
-own block table ``[slots, pages per sequence]``.  A group with a window gives
+own block table ``[slots, pages per sequence]``.  A group with a window or chunks gives
 pages back as soon as no later query can see any key in them; every group
 gives all of a request's pages back when the request ends.
 
@@ -147,10 +147,7 @@ class CacheManager:
 
     def _first_needed_page(self, group: CacheGroup, first_query_pos: int) -> int:
         """Lowest logical page holding a key that a query at ``first_query_pos`` or later sees."""
-        if group.spec.window is None:
-            return 0
-        first_key = max(0, first_query_pos - group.spec.window + 1)
-        return first_key // self.page_size
+        return group.spec.first_key(first_query_pos) // self.page_size
 
     def pages_needed(self, slot: int, n_new: int) -> list[int]:
         """Per group, how many new pages ``reserve(slot, n_new)`` would take."""
@@ -202,11 +199,11 @@ class CacheManager:
 
     def commit(self, slot: int, n_new: int) -> None:
         """The step that used ``reserve(slot, n_new)`` has been issued: count the tokens
-        and give back pages that a window has passed."""
+        and give back pages that a window or a chunk has passed."""
         self.num_tokens[slot] += n_new
         cur = int(self.num_tokens[slot])
         for g in self.groups:
-            if g.spec.window is None:
+            if not g.spec.bounded:
                 continue
             keep_from = self._first_needed_page(g, cur)
             lo = int(g.first_page[slot])

@@ -16,6 +16,7 @@ from .lebedra import LebedraConfig
 from .porovik import PorovikConfig
 from .fikevik import FikevikConfig
 from .soporax import SoporaxConfig
+from .vebotar import VebotarConfig
 
 __all__ = [
     "Architecture",
@@ -26,6 +27,7 @@ __all__ = [
     "PorovikConfig",
     "FikevikConfig",
     "SoporaxConfig",
+    "VebotarConfig",
     "ModelConfig",
     "load_config",
     "parse_config",

@@ -8,6 +8,13 @@
 //   head_scale  : a further factor of the score per head, from a table            (absent: 1)
 //   window      : a query at i sees the keys j with 0 <= i - j < window            (0: all keys j <= i);
 //                 pages that lie wholly before a block's window are never looked up (the cache gives them back)
+//   chunk       : a query at i sees the keys j <= i of its own chunk, floor(j / chunk) = floor(i / chunk), chunks counted
+//                 from the sequence's first token (0: no chunks); pages of earlier chunks are never looked up
+//   maps        : 2: differential attention.  A head has two query vectors and a key/value head two keys a token, side by
+//                 side ([map 1 | map 2], dk entries each; the cache row is [key 1 | key 2 | value]); each map is a softmax
+//                 of its own over the same values, and the head's result is o = a_1 - lambda a_2 (lambda: one device
+//                 scalar), then o / sqrt(mean(o^2) + eps) over its dv columns times a constant.  A block holds both maps
+//                 of its rows, so keys and values are fetched once for the two.
 //   sink        : one more term exp(sink_h) in the softmax's denominator, a table with one entry a head; it
 //                 has no key and no value and is not scaled                       (absent: a plain softmax)
 //   out         = softmax(score) V * sigmoid(gate)                             (gate absent: no gate); the gate's
@@ -57,6 +64,9 @@ struct BiasAttnParams {
   float* part_o;
   float* part_ml;
   const float* sink;  // [n_heads] or null
+  int chunk;           // 0: none
+  const float* diff_lambda;  // two maps: the factor of the second (device scalar)
+  float diff_eps, diff_mul;  // and what the difference's root mean square adds inside, and its constant factor
   int gate_per_head;  // the gate holds one logit a (token, head): [tokens, ldg], head h at column h
 };
 
@@ -65,6 +75,13 @@ __device__ __forceinline__ const float* bias_gate_row(const BiasAttnParams& p, i
   stride = p.gate_per_head ? 0 : 1;
   if (p.gate == nullptr) return nullptr;
   return p.gate + (size_t)tok * p.ldg + (p.gate_per_head ? (size_t)head : (size_t)head * p.dv);
+}
+
+// The first key that a query at `pos` sees.
+__device__ __forceinline__ int bias_first_seen(const BiasAttnParams& p, int pos) {
+  int lo = p.window > 0 ? pos - p.window + 1 : 0;
+  if (p.chunk > 0) lo = max(lo, pos / p.chunk * p.chunk);
+  return max(lo, 0);
 }
 
 }  // namespace rl
@@ -76,9 +93,12 @@ namespace rl {
 // LPR lanes share a row (their keys tx + LPR b, their value columns tx + LPR c), RPT rows a thread: a block has
 // (BA_THREADS / LPR) * RPT rows.  Prompt tiles run 8 lanes x 2 rows (32 rows); a decoded token has only its
 // group's heads as rows, so its blocks run 16 or 32 lanes a row (8 or 4 rows) and every thread has work.
-template <typename T, int LPR, int RPT, int DVC, typename TOut>
+// With two maps the first half of the rows are (token, head) pairs of map 1, the second half the same pairs of map 2.
+template <typename T, int LPR, int RPT, int DVC, typename TOut, int MAPS>
 __global__ __launch_bounds__(BA_THREADS) void bias_attn_kernel(const BiasAttnParams p) {
   constexpr int ROWS = BA_THREADS / LPR * RPT, KPT = BA_KEYS / LPR;
+  constexpr int PAIRS = ROWS / MAPS;  // (token, head) pairs
+  static_assert(PAIRS % RPT == 0, "a thread's rows belong to one map");
   extern __shared__ __align__(16) float ba_s[];
   pdl_begin();
   const int subs = p.tile_tokens / p.tokens_per_block;
@@ -104,7 +124,8 @@ __global__ __launch_bounds__(BA_THREADS) void bias_attn_kernel(const BiasAttnPar
   const int hb0 = blockIdx.z * p.heads_per_block;
   const int HB = p.heads_per_block;
   const int dk = p.dk, dv = p.dv;
-  const int ldq_s = dk | 1, ldk_s = dk | 1, ldv_s = LPR * DVC;
+  const int kd = MAPS * dk;  // a token's keys
+  const int ldq_s = dk | 1, ldk_s = kd | 1, ldv_s = LPR * DVC;
   float* Qs = ba_s;                        // [ROWS][ldq_s]
   float* Ks = Qs + ROWS * ldq_s;           // [BA_KEYS][ldk_s]
   float* Vs = Ks + BA_KEYS * ldk_s;        // [BA_KEYS][ldv_s]
@@ -113,20 +134,22 @@ __global__ __launch_bounds__(BA_THREADS) void bias_attn_kernel(const BiasAttnPar
   const int ty = tid / LPR, tx = tid % LPR;
   // queries
   for (int r = warp; r < ROWS; r += BA_THREADS / 32) {
-    const int tl = r / HB, hl = r - tl * HB;
+    const int pr = r % PAIRS, tl = pr / HB, hl = pr - tl * HB;
     const bool ok = tl < n_tok && hb0 + hl < hg;
-    const float* src = p.q + (size_t)(t_begin + first + tl) * p.ldq + (size_t)(g * hg + hb0 + hl) * dk;
+    const float* src = p.q + (size_t)(t_begin + first + tl) * p.ldq + (size_t)(g * hg + hb0 + hl) * kd + (r / PAIRS) * dk;
     for (int d = lane; d < dk; d += 32) Qs[r * ldq_s + d] = ok ? src[d] : 0.f;
   }
-  int row_pos[RPT], row_head[RPT];
+  int row_pos[RPT], row_lo[RPT], row_head[RPT];
   float row_mul[RPT], row_slope[RPT], m[RPT], l[RPT];
   bool row_ok[RPT];
+  const int map = ty * RPT / PAIRS;  // of the thread's rows
   float acc[RPT][DVC];
 #pragma unroll
   for (int a = 0; a < RPT; ++a) {
-    const int r = ty * RPT + a, tl = r / HB, hl = r - tl * HB;
+    const int r = ty * RPT + a - map * PAIRS, tl = r / HB, hl = r - tl * HB;
     row_ok[a] = tl < n_tok && hb0 + hl < hg;
     row_pos[a] = pos0 + tl;
+    row_lo[a] = bias_first_seen(p, row_pos[a]);
     row_head[a] = g * hg + hb0 + hl;
     float temp = 1.0f;
     if (p.temp_every > 0) temp = 1.0f + p.temp_coef * logf((float)((row_pos[a] + 1) / p.temp_every + 1));
@@ -139,7 +162,7 @@ __global__ __launch_bounds__(BA_THREADS) void bias_attn_kernel(const BiasAttnPar
     for (int c = 0; c < DVC; ++c) acc[a][c] = 0.f;
   }
   const int last_pos = pos0 + n_tok - 1;
-  const int first_seen = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;  // the earliest key any row of the block sees
+  const int first_seen = bias_first_seen(p, pos0);  // the earliest key any row of the block sees
   const T* pool = reinterpret_cast<const T*>(p.pool);
   const int* table = p.block_table + (size_t)slot * p.ldt;
   // Where each key of a tile lies (null: beyond the block's last position, or no page): looked up by one
@@ -162,7 +185,7 @@ __global__ __launch_bounds__(BA_THREADS) void bias_attn_kernel(const BiasAttnPar
     }
   };
   constexpr int EV = 16 / (int)sizeof(T);  // elements of a 16-byte piece
-  const bool vec = dk % EV == 0 && dv % EV == 0 && p.row % EV == 0 && p.v_at % EV == 0 &&
+  const bool vec = kd % EV == 0 && dv % EV == 0 && p.row % EV == 0 && p.v_at % EV == 0 &&
                    (reinterpret_cast<uintptr_t>(p.pool) & 15) == 0;
   for (int i = tid; i < BA_KEYS * ldv_s; i += BA_THREADS) Vs[i] = 0.f;  // the fill beyond dv stays zero
   int j_begin = first_seen / BA_KEYS * BA_KEYS, j_end = last_pos + 1;  // the keys this block walks
@@ -177,7 +200,7 @@ __global__ __launch_bounds__(BA_THREADS) void bias_attn_kernel(const BiasAttnPar
   for (int j0 = j_begin; j0 < j_end; j0 += BA_KEYS, buf ^= 1) {
     __syncthreads();  // the tile before has been used; this tile's places (and, the first time, the queries) are known
     if (vec) {
-      const int kp = dk / EV, vp = dv / EV, per_key = kp + vp;
+      const int kp = kd / EV, vp = dv / EV, per_key = kp + vp;
 #pragma unroll 4
       for (int i = tid; i < BA_KEYS * per_key; i += BA_THREADS) {
         const int jj = i / per_key, piece = i - jj * per_key;
@@ -192,14 +215,14 @@ __global__ __launch_bounds__(BA_THREADS) void bias_attn_kernel(const BiasAttnPar
         for (int x = 0; x < EV; ++x) dst[x] = to_f32(e[x]);
       }
     } else {
-      const int per_key = dk + dv;
+      const int per_key = kd + dv;
 #pragma unroll 4
       for (int i = tid; i < BA_KEYS * per_key; i += BA_THREADS) {
         const int jj = i / per_key, c = i - jj * per_key;
         const T* src = key_src[buf][jj];
-        const bool is_v = c >= dk;
-        const float val = src != nullptr ? to_f32(src[is_v ? p.v_at + c - dk : c]) : 0.f;
-        if (is_v) Vs[jj * ldv_s + c - dk] = val;
+        const bool is_v = c >= kd;
+        const float val = src != nullptr ? to_f32(src[is_v ? p.v_at + c - kd : c]) : 0.f;
+        if (is_v) Vs[jj * ldv_s + c - kd] = val;
         else Ks[jj * ldk_s + c] = val;
       }
     }
@@ -207,7 +230,7 @@ __global__ __launch_bounds__(BA_THREADS) void bias_attn_kernel(const BiasAttnPar
     __syncthreads();
     float s[RPT][KPT] = {};
     const float* q0 = Qs + (ty * RPT) * ldq_s;
-    const float* kb = Ks + tx * ldk_s;
+    const float* kb = Ks + tx * ldk_s + map * dk;
 #pragma unroll 4
     for (int d = 0; d < dk; ++d) {
       float qa[RPT];
@@ -226,7 +249,7 @@ __global__ __launch_bounds__(BA_THREADS) void bias_attn_kernel(const BiasAttnPar
 #pragma unroll
       for (int b = 0; b < KPT; ++b) {
         const int j = j0 + tx + LPR * b;
-        const bool see = row_ok[a] && j <= row_pos[a] && (p.window <= 0 || row_pos[a] - j < p.window);
+        const bool see = row_ok[a] && j <= row_pos[a] && j >= row_lo[a];
         s[a][b] = see ? s[a][b] * row_mul[a] - row_slope[a] * (float)(row_pos[a] - j) : -CUDART_INF_F;
         tile_max = fmaxf(tile_max, s[a][b]);
       }
@@ -268,7 +291,7 @@ __global__ __launch_bounds__(BA_THREADS) void bias_attn_kernel(const BiasAttnPar
 #pragma unroll
     for (int a = 0; a < RPT; ++a) {
       if (!row_ok[a]) continue;
-      const size_t at = ((size_t)dec * p.n_heads + row_head[a]) * p.n_splits + split;
+      const size_t at = (((size_t)dec * p.n_heads + row_head[a]) * MAPS + map) * p.n_splits + split;
 #pragma unroll
       for (int c = 0; c < DVC; ++c)
         if (tx + LPR * c < dv) p.part_o[at * dv + tx + LPR * c] = acc[a][c];
@@ -279,21 +302,57 @@ __global__ __launch_bounds__(BA_THREADS) void bias_attn_kernel(const BiasAttnPar
     }
     return;
   }
+  if constexpr (MAPS == 2) {
+    // the second map's rows pass their results through shared memory to the threads of the first map's
+    float* second = ba_s;  // [PAIRS][LPR * DVC]: queries, keys and values have been used
+    __syncthreads();
+    if (map == 1) {
 #pragma unroll
-  for (int a = 0; a < RPT; ++a) {
-    if (!row_ok[a]) continue;
-    const int tok = t_begin + first + (ty * RPT + a) / HB;
-    const float inv = 1.0f / (l[a] + (p.sink != nullptr ? expf(p.sink[row_head[a]] - m[a]) : 0.f));
-    TOut* o = reinterpret_cast<TOut*>(p.out) + (size_t)tok * p.ldo + (size_t)row_head[a] * dv;
-    int gs;
-    const float* gr = bias_gate_row(p, tok, row_head[a], gs);
+      for (int a = 0; a < RPT; ++a) {
+        const float inv = row_ok[a] ? 1.0f / l[a] : 0.f;
 #pragma unroll
-    for (int c = 0; c < DVC; ++c) {
-      const int col = tx + LPR * c;
-      if (col < dv) {
-        float v = acc[a][c] * inv;
-        if (gr != nullptr) v *= 1.0f / (1.0f + expf(-gr[col * gs]));
-        o[col] = from_f32<TOut>(v);
+        for (int c = 0; c < DVC; ++c) second[(ty * RPT + a - PAIRS) * (LPR * DVC) + tx + LPR * c] = acc[a][c] * inv;
+      }
+    }
+    __syncthreads();
+    if (map == 1) return;
+    const float lambda = *p.diff_lambda;
+#pragma unroll
+    for (int a = 0; a < RPT; ++a) {
+      const float inv = row_ok[a] ? 1.0f / l[a] : 0.f;
+      float ss = 0.f;
+#pragma unroll
+      for (int c = 0; c < DVC; ++c) {  // columns beyond dv are zero in both maps
+        acc[a][c] = fmaf(-lambda, second[(ty * RPT + a) * (LPR * DVC) + tx + LPR * c], acc[a][c] * inv);
+        ss = fmaf(acc[a][c], acc[a][c], ss);
+      }
+#pragma unroll
+      for (int o = 1; o < LPR; o <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      const float mul = p.diff_mul / sqrtf(ss / (float)dv + p.diff_eps);
+      if (!row_ok[a]) continue;
+      const int tok = t_begin + first + (ty * RPT + a) / HB;
+      TOut* o = reinterpret_cast<TOut*>(p.out) + (size_t)tok * p.ldo + (size_t)row_head[a] * dv;
+#pragma unroll
+      for (int c = 0; c < DVC; ++c)
+        if (tx + LPR * c < dv) o[tx + LPR * c] = from_f32<TOut>(acc[a][c] * mul);
+    }
+  } else {
+#pragma unroll
+    for (int a = 0; a < RPT; ++a) {
+      if (!row_ok[a]) continue;
+      const int tok = t_begin + first + (ty * RPT + a) / HB;
+      const float inv = 1.0f / (l[a] + (p.sink != nullptr ? expf(p.sink[row_head[a]] - m[a]) : 0.f));
+      TOut* o = reinterpret_cast<TOut*>(p.out) + (size_t)tok * p.ldo + (size_t)row_head[a] * dv;
+      int gs;
+      const float* gr = bias_gate_row(p, tok, row_head[a], gs);
+#pragma unroll
+      for (int c = 0; c < DVC; ++c) {
+        const int col = tx + LPR * c;
+        if (col < dv) {
+          float v = acc[a][c] * inv;
+          if (gr != nullptr) v *= 1.0f / (1.0f + expf(-gr[col * gs]));
+          o[col] = from_f32<TOut>(v);
+        }
       }
     }
   }
@@ -336,6 +395,53 @@ __global__ __launch_bounds__(128) void bias_attn_merge_kernel(const BiasAttnPara
   }
 }
 
+// The same for two maps: a warp a (decoded request, head) puts each map's parts together, then forms the difference and
+// brings it to unit root mean square.  dv <= 256: eight columns a lane.
+template <typename TOut>
+__global__ __launch_bounds__(128) void bias_attn_merge_maps_kernel(const BiasAttnParams p) {
+  pdl_begin();
+  const int dec = blockIdx.x, req = p.decode_reqs[dec];
+  if (p.slots[req] < 0) return;
+  const int tok = p.q_start[req], dv = p.dv;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int head = blockIdx.y * 4 + warp;
+  if (head >= p.n_heads) return;
+  float r[8];
+#pragma unroll
+  for (int c = 0; c < 8; ++c) r[c] = 0.f;
+  const float lambda = *p.diff_lambda;
+#pragma unroll
+  for (int map = 0; map < 2; ++map) {
+    const size_t at = (((size_t)dec * p.n_heads + head) * 2 + map) * p.n_splits;
+    const float ms = lane < p.n_splits ? p.part_ml[2 * (at + lane)] : -CUDART_INF_F;
+    const float ls = lane < p.n_splits ? p.part_ml[2 * (at + lane) + 1] : 0.f;
+    const float M = warp_max(ms);
+    const float w = ms == -CUDART_INF_F ? 0.f : expf(ms - M);
+    float L = 0.f;
+    for (int s = 0; s < p.n_splits; ++s) L = fmaf(__shfl_sync(0xffffffffu, ls, s), __shfl_sync(0xffffffffu, w, s), L);
+    const float factor = (map == 0 ? 1.0f : -lambda) / L;
+#pragma unroll
+    for (int c = 0; c < 8; ++c) {
+      const int col = c * 32 + lane;
+      if (c * 32 >= dv) break;
+      float acc = 0.f;
+      for (int s = 0; s < p.n_splits; ++s) {
+        const float ws = __shfl_sync(0xffffffffu, w, s);
+        if (col < dv && ws != 0.f) acc = fmaf(p.part_o[(at + s) * dv + col], ws, acc);
+      }
+      r[c] = fmaf(acc, factor, r[c]);
+    }
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int c = 0; c < 8; ++c) ss = fmaf(r[c], r[c], ss);
+  const float mul = p.diff_mul / sqrtf(warp_sum(ss) / (float)dv + p.diff_eps);
+  TOut* o = reinterpret_cast<TOut*>(p.out) + (size_t)tok * p.ldo + (size_t)head * dv;
+#pragma unroll
+  for (int c = 0; c < 8; ++c)
+    if (c * 32 + lane < dv) o[c * 32 + lane] = from_f32<TOut>(r[c] * mul);
+}
+
 // mix: 0 values as they are; 1 also left in v_src (this layer is the source); 2 mixed with v_src by *lambda.
 template <typename T>
 __global__ void bias_kv_store_kernel(const float* __restrict__ k, long ldk, const float* __restrict__ v, long ldv,
@@ -371,12 +477,12 @@ __global__ void bias_kv_store_kernel(const float* __restrict__ k, long ldk, cons
   }
 }
 
-template <typename T, int LPR, int RPT, int DVC, typename TOut>
+template <typename T, int LPR, int RPT, int DVC, typename TOut, int MAPS>
 static void launch_bias_attn(const BiasAttnParams& p, dim3 grid, cudaStream_t stream) {
   constexpr int ROWS = BA_THREADS / LPR * RPT;
-  const size_t smem = ((size_t)ROWS * (p.dk | 1) + (size_t)BA_KEYS * (p.dk | 1) + (size_t)BA_KEYS * LPR * DVC +
+  const size_t smem = ((size_t)ROWS * (p.dk | 1) + (size_t)BA_KEYS * (MAPS * p.dk | 1) + (size_t)BA_KEYS * LPR * DVC +
                        (size_t)ROWS * (BA_KEYS + 1)) * sizeof(float);
-  auto kernel = bias_attn_kernel<T, LPR, RPT, DVC, TOut>;
+  auto kernel = bias_attn_kernel<T, LPR, RPT, DVC, TOut, MAPS>;
   if (smem > 48 * 1024) {
     static bool raised = false;
     if (!raised) {
@@ -388,30 +494,35 @@ static void launch_bias_attn(const BiasAttnParams& p, dim3 grid, cudaStream_t st
 }
 
 // rows: 32 (prompt tiles, and decoded tokens of large groups), 8 or 4 (decoded tokens)
-template <typename T, typename TOut>
+template <typename T, typename TOut, int MAPS>
 static void dispatch_bias_attn(const BiasAttnParams& p, int rows, dim3 grid, cudaStream_t stream) {
   if (rows == 4) {
-    if (p.dv <= 64) launch_bias_attn<T, 32, 1, 2, TOut>(p, grid, stream);
-    else launch_bias_attn<T, 32, 1, 8, TOut>(p, grid, stream);
+    if (p.dv <= 64) launch_bias_attn<T, 32, 1, 2, TOut, MAPS>(p, grid, stream);
+    else if (MAPS == 2 && p.dv <= 128) launch_bias_attn<T, 32, 1, 4, TOut, MAPS>(p, grid, stream);
+    else launch_bias_attn<T, 32, 1, 8, TOut, MAPS>(p, grid, stream);
   } else if (rows == 8) {
-    if (p.dv <= 64) launch_bias_attn<T, 16, 1, 4, TOut>(p, grid, stream);
-    else launch_bias_attn<T, 16, 1, 16, TOut>(p, grid, stream);
+    if (p.dv <= 64) launch_bias_attn<T, 16, 1, 4, TOut, MAPS>(p, grid, stream);
+    else if (MAPS == 2 && p.dv <= 128) launch_bias_attn<T, 16, 1, 8, TOut, MAPS>(p, grid, stream);
+    else launch_bias_attn<T, 16, 1, 16, TOut, MAPS>(p, grid, stream);
   } else {
-    if (p.dv <= 32) launch_bias_attn<T, 8, 2, 4, TOut>(p, grid, stream);
-    else if (p.dv <= 64) launch_bias_attn<T, 8, 2, 8, TOut>(p, grid, stream);
-    else if (p.dv <= 128) launch_bias_attn<T, 8, 2, 16, TOut>(p, grid, stream);
-    else launch_bias_attn<T, 8, 2, 32, TOut>(p, grid, stream);
+    if (p.dv <= 32) launch_bias_attn<T, 8, 2, 4, TOut, MAPS>(p, grid, stream);
+    else if (p.dv <= 64) launch_bias_attn<T, 8, 2, 8, TOut, MAPS>(p, grid, stream);
+    else if (p.dv <= 128) launch_bias_attn<T, 8, 2, 16, TOut, MAPS>(p, grid, stream);
+    else launch_bias_attn<T, 8, 2, 32, TOut, MAPS>(p, grid, stream);
   }
 }
 
-static void dispatch_bias_attn_types(int cache_dtype, int out_dtype, const BiasAttnParams& p, int rows, dim3 grid,
+static void dispatch_bias_attn_types(int cache_dtype, int out_dtype, int maps, const BiasAttnParams& p, int rows, dim3 grid,
                                      cudaStream_t stream) {
-  if (cache_dtype == RL_F32) {
-    if (out_dtype == RL_F32) dispatch_bias_attn<float, float>(p, rows, grid, stream);
-    else dispatch_bias_attn<float, __nv_bfloat16>(p, rows, grid, stream);
+  if (maps == 2) {  // cache and output of one type
+    if (cache_dtype == RL_F32) dispatch_bias_attn<float, float, 2>(p, rows, grid, stream);
+    else dispatch_bias_attn<__nv_bfloat16, __nv_bfloat16, 2>(p, rows, grid, stream);
+  } else if (cache_dtype == RL_F32) {
+    if (out_dtype == RL_F32) dispatch_bias_attn<float, float, 1>(p, rows, grid, stream);
+    else dispatch_bias_attn<float, __nv_bfloat16, 1>(p, rows, grid, stream);
   } else {
-    if (out_dtype == RL_F32) dispatch_bias_attn<__nv_bfloat16, float>(p, rows, grid, stream);
-    else dispatch_bias_attn<__nv_bfloat16, __nv_bfloat16>(p, rows, grid, stream);
+    if (out_dtype == RL_F32) dispatch_bias_attn<__nv_bfloat16, float, 1>(p, rows, grid, stream);
+    else dispatch_bias_attn<__nv_bfloat16, __nv_bfloat16, 1>(p, rows, grid, stream);
   }
 }
 
@@ -421,11 +532,11 @@ static void dispatch_bias_attn_types(int cache_dtype, int out_dtype, const BiasA
 // (on by default; sizes that cannot be copied in 16-byte pieces never take it).
 RL_EXPORT void rl_bias_attention_async(int on) { rl::BIAS_ATTENTION_ASYNC = on != 0; }
 
-// How the `rows` rows of a prompt tile's block (32: the CUDA-core kernel; 64: the tensor-core kernel) are cut
-// into tokens and heads for `heads_per_group` query heads a key/value head: heads a block (at most `rows`) and
+// How the `rows` (token, head) pairs of a prompt tile's block (32: the CUDA-core kernel; 64: the tensor-core kernel; 16:
+// the CUDA-core kernel with two maps, whose 32 rows are 16 pairs) are cut into tokens and heads for `heads_per_group` query heads a key/value head: heads a block (at most `rows`) and
 // tokens a block (a power of two, at most `rows`).
 RL_EXPORT int rl_bias_attention_shape(int heads_per_group, int rows, int* heads_per_block, int* tokens_per_block) {
-  if (heads_per_group <= 0 || (rows != rl::BA_ROWS && rows != rl::BM_ROWS)) return -2;
+  if (heads_per_group <= 0 || (rows != rl::BA_ROWS && rows != rl::BA_ROWS / 2 && rows != rl::BM_ROWS)) return -2;
   const int hb = heads_per_group < rows ? heads_per_group : rows;
   int tt = 1;
   while (tt * 2 * hb <= rows) tt *= 2;
@@ -439,6 +550,9 @@ RL_EXPORT int rl_bias_attention_shape(int heads_per_group, int rows, int* heads_
 // tensor_cores: prompt tiles go to `bias_attn_mma_kernel` where the types and sizes allow (64 rows a block: the
 // tiles must then be cut as rl_bias_attention_shape(.., 64, ..) says).
 // sink: float32 [heads] or null; gate_per_head: the gate's rows hold one logit a head, not one a value column.
+// chunk: 0, or the chunk's size.  maps: 1, or 2 (differential attention: see the top; q holds two vectors a head, the
+// cache rows two keys; the cache's and the output's type are one; no gate, no sink; diff_lambda a device scalar; part_o
+// and part_ml have an entry a map: [n_decode * heads * 2 * n_splits, ..]).
 // tiles: (request, first new token) of portions cut every `tile_tokens` tokens (a multiple of the tokens a
 // block takes); decode_reqs: the requests that bring one token.  cache_dtype: the pool's element type;
 // out_dtype: that of out.
@@ -449,15 +563,19 @@ RL_EXPORT int rl_bias_attention(int cache_dtype, int out_dtype, const float* q, 
                                 int dv, int v_at, int row, int page_size, int max_pages, float scale, float temp_coef,
                                 int temp_every, const float* slopes, int* status, int n_splits, float* part_o,
                                 float* part_ml, int tensor_cores, int window, const float* head_scale,
-                                const float* sink, int gate_per_head, cudaStream_t stream) {
+                                const float* sink, int gate_per_head, int chunk, int maps, const float* diff_lambda,
+                                float diff_eps, float diff_mul, cudaStream_t stream) {
   if (n_tiles <= 0 && n_decode <= 0) return 0;
-  if (n_heads <= 0 || n_kv <= 0 || n_heads % n_kv || dk <= 0 || dk > 256 || dv <= 0 || dv > 256 || v_at < dk ||
-      v_at + dv > row || n_kv > 65535 || window < 0)
+  if (n_heads <= 0 || n_kv <= 0 || n_heads % n_kv || dk <= 0 || dk > 256 || dv <= 0 || dv > 256 || maps < 1 || maps > 2 ||
+      v_at < maps * dk || v_at + dv > row || n_kv > 65535 || window < 0 || chunk < 0)
     return -2;
+  if (maps == 2 && (diff_lambda == nullptr || gate != nullptr || sink != nullptr || cache_dtype != out_dtype)) return -5;
   // prompt tiles on the tensor cores: bfloat16 cache and output, per-head sizes up to 128
-  const bool mma = tensor_cores && cache_dtype == RL_BF16 && out_dtype == RL_BF16 && dk <= 128 && dv <= 128;
+  // (two maps only in the form whose tiles are copied in 16-byte pieces)
+  const bool mma = tensor_cores && cache_dtype == RL_BF16 && out_dtype == RL_BF16 && dk <= 128 && dv <= 128 &&
+                   (maps == 1 || (dk % 8 == 0 && dv % 8 == 0 && v_at % 8 == 0 && row % 8 == 0 && ((uintptr_t)pool & 15) == 0));
   int hb, tt;
-  rl_bias_attention_shape(n_heads / n_kv, mma ? rl::BM_ROWS : rl::BA_ROWS, &hb, &tt);
+  rl_bias_attention_shape(n_heads / n_kv, mma ? rl::BM_ROWS : rl::BA_ROWS / maps, &hb, &tt);
   if (n_tiles > 0 && (tile_tokens < tt || tile_tokens % tt)) return -3;
   if (n_tiles <= 0) tile_tokens = tt;
   if (n_splits < 1 || n_splits > 32 || (n_splits > 1 && (part_o == nullptr || part_ml == nullptr))) return -4;
@@ -466,25 +584,28 @@ RL_EXPORT int rl_bias_attention(int cache_dtype, int out_dtype, const float* q, 
   rl::BiasAttnParams p{q, ldq, gate, ldg, pool, block_table, ldt, q_start, kv_len, slots, tiles, decode_reqs, out, ldo,
                        n_heads, n_kv, dk, dv, v_at, row, page_size, max_pages, n_tiles > 0 ? n_tiles : 0, tile_tokens,
                        tt, hb, 0, scale, temp_coef, temp_every, slopes, status, window, head_scale, 1, part_o, part_ml,
-                       sink, gate_per_head != 0};
+                       sink, chunk, diff_lambda, diff_eps, diff_mul, gate_per_head != 0};
   if (p.n_tiles > 0) {  // the prompt portions: 32 or 64 rows a block, cut into tokens and heads as rl_bias_attention_shape says
     const dim3 grid(p.n_tiles * (tile_tokens / tt), n_kv, (hg + hb - 1) / hb);
-    if (mma) rl::dispatch_bias_attn_mma(p, grid, stream);
-    else rl::dispatch_bias_attn_types(cache_dtype, out_dtype, p, 32, grid, stream);
+    if (mma) rl::dispatch_bias_attn_mma(p, maps, grid, stream);
+    else rl::dispatch_bias_attn_types(cache_dtype, out_dtype, maps, p, 32, grid, stream);
   }
   if (n_decode > 0) {  // the decoded tokens: a block's rows are heads of one group, 4, 8 or 32 of them
-    const int rows = hg <= 4 ? 4 : (hg <= 8 ? 8 : 32);
+    const int rows = hg * maps <= 4 ? 4 : (hg * maps <= 8 ? 8 : 32);
     p.n_tiles = 0;
     p.n_decode = n_decode;
     p.n_splits = n_splits;
     p.tokens_per_block = p.tile_tokens = 1;
-    p.heads_per_block = hg < rows ? hg : rows;
-    rl::dispatch_bias_attn_types(cache_dtype, out_dtype, p, rows,
+    p.heads_per_block = hg < rows / maps ? hg : rows / maps;
+    rl::dispatch_bias_attn_types(cache_dtype, out_dtype, maps, p, rows,
                                  dim3(n_decode * n_splits, n_kv, (hg + p.heads_per_block - 1) / p.heads_per_block), stream);
   }
   if (n_splits > 1) {
     const dim3 mg(p.n_decode, (n_heads + 3) / 4);
-    if (out_dtype == RL_F32) rl::launch_pdl(rl::bias_attn_merge_kernel<float>, mg, 128, 0, stream, p);
+    if (maps == 2) {
+      if (out_dtype == RL_F32) rl::launch_pdl(rl::bias_attn_merge_maps_kernel<float>, mg, 128, 0, stream, p);
+      else rl::launch_pdl(rl::bias_attn_merge_maps_kernel<__nv_bfloat16>, mg, 128, 0, stream, p);
+    } else if (out_dtype == RL_F32) rl::launch_pdl(rl::bias_attn_merge_kernel<float>, mg, 128, 0, stream, p);
     else rl::launch_pdl(rl::bias_attn_merge_kernel<__nv_bfloat16>, mg, 128, 0, stream, p);
   }
   RL_CHECK_LAUNCH();
@@ -522,7 +643,10 @@ namespace rl {
 //     multiplied by a weight the heads share (q_norm / k_norm; absent: left as they are, or with `unit_qk`
 //     divided by the root mean square and no weight), then the first
 //     `rot_dims` entries turned, entry 2i with entry 2i + 1, by the angle position * freq[i];
+//     cosines and sines times `rot_mult`;
 //   values: each head's entries divided by their root mean square, no weight (unit_values; else untouched).
+// `maps` query vectors a head and keys a key/value head (each normalised and turned by itself), a token's keys of one
+// key/value head side by side in the cache row.  k null: queries alone (a layer that reads another layer's cache).
 // Angles are formed and evaluated in float32.  With a cache target the keys and values go into their pages on the
 // way (as `bias_kv_store_kernel` would put them) and are not written back.
 // Where the keys and values of a step go when this kernel also writes the cache (fused: the store kernel's work
@@ -543,8 +667,8 @@ __global__ __launch_bounds__(128) void qkv_norm_rotate_kernel(float* __restrict_
                                                               const float* __restrict__ k_norm,
                                                               const float* __restrict__ freq,
                                                               const int* __restrict__ positions, int n_tokens,
-                                                              int n_heads, int n_kv, int dk, int dv, int rot_dims,
-                                                              int unit_values, int unit_qk, float eps,
+                                                              int n_heads, int n_kv, int maps, int dk, int dv, int rot_dims,
+                                                              float rot_mult, int unit_values, int unit_qk, float eps,
                                                               const QkvCacheTarget c) {
   pdl_begin();
   const int tok = blockIdx.x;
@@ -553,7 +677,8 @@ __global__ __launch_bounds__(128) void qkv_norm_rotate_kernel(float* __restrict_
   const int ipos = positions[tok];
   const float pos = (float)ipos;
   const bool store = c.pool != nullptr;
-  const int units = n_heads + n_kv + ((unit_values || store) ? n_kv : 0);
+  const int nq = n_heads * maps, nk = k != nullptr ? n_kv * maps : 0;  // vectors of dk entries
+  const int units = nq + nk + ((unit_values || store) ? n_kv : 0);
   // the token's place in the cache: a row of its page a key/value head (null: a padding row, or no page)
   T* cache_row = nullptr;
   long head_step = 0;
@@ -573,14 +698,22 @@ __global__ __launch_bounds__(128) void qkv_norm_rotate_kernel(float* __restrict_
   }
   // the token's angles are the same for all its heads: their sines and cosines once a block
   __shared__ float2 turn[128];
-  for (int i = threadIdx.x; 2 * i < rot_dims; i += blockDim.x) sincosf(pos * freq[i], &turn[i].y, &turn[i].x);
+  for (int i = threadIdx.x; 2 * i < rot_dims; i += blockDim.x) {
+    float sn, cs;
+    sincosf(pos * freq[i], &sn, &cs);
+    turn[i] = make_float2(cs * rot_mult, sn * rot_mult);
+  }
   __syncthreads();
   for (int u = blockIdx.y * n_warps + warp; u < units; u += n_warps * gridDim.y) {
-    if (u < n_heads + n_kv) {
-      const bool is_q = u < n_heads;
-      float* e = is_q ? q + (size_t)tok * ldq + (size_t)u * dk : k + (size_t)tok * ldk + (size_t)(u - n_heads) * dk;
+    if (u < nq + nk) {
+      const bool is_q = u < nq;
+      float* e = is_q ? q + (size_t)tok * ldq + (size_t)u * dk : k + (size_t)tok * ldk + (size_t)(u - nq) * dk;
       const float* w = is_q ? q_norm : k_norm;
-      T* to_cache = (!is_q && cache_row != nullptr) ? cache_row + (size_t)(u - n_heads) * head_step : nullptr;
+      T* to_cache = nullptr;
+      if (!is_q && cache_row != nullptr) {
+        const int g = (u - nq) / maps;
+        to_cache = cache_row + (size_t)g * head_step + (size_t)(u - nq - g * maps) * dk;
+      }
       const bool in_place = is_q || !store;
       float r = 1.0f;
       if (w != nullptr || unit_qk) {
@@ -611,7 +744,7 @@ __global__ __launch_bounds__(128) void qkv_norm_rotate_kernel(float* __restrict_
         }
       }
     } else {
-      const int g = u - n_heads - n_kv;
+      const int g = u - nq - nk;
       float* e = v + (size_t)tok * ldv + (size_t)g * dv;
       float r = 1.0f;
       if (unit_values) {
@@ -639,28 +772,30 @@ __global__ __launch_bounds__(128) void qkv_norm_rotate_kernel(float* __restrict_
 // their pages (the value at entry v_at of a row) instead of back in place, as rl_bias_kv_store would put them.
 RL_EXPORT int rl_qkv_norm_rotate(float* q, long ldq, float* k, long ldk, float* v, long ldv, const float* q_norm,
                                  const float* k_norm, const float* freq, const int* positions, int n_tokens, int n_heads,
-                                 int n_kv, int dk, int dv, int rot_dims, int unit_values, int unit_qk, float eps,
-                                 int cache_dtype, void* pool, const int* block_table, long ldt, const int* req_of_token,
+                                 int n_kv, int maps, int dk, int dv, int rot_dims, float rot_mult, int unit_values,
+                                 int unit_qk, float eps, int cache_dtype, void* pool, const int* block_table, long ldt, const int* req_of_token,
                                  const int* slots, int v_at, int row, int page_size, int max_pages, int* status,
                                  cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
-  if (n_heads <= 0 || n_kv <= 0 || dk <= 0 || dv <= 0 || rot_dims < 0 || rot_dims % 2 || rot_dims > dk ||
+  if (n_heads <= 0 || n_kv <= 0 || maps < 1 || dk <= 0 || dv <= 0 || rot_dims < 0 || rot_dims % 2 || rot_dims > dk ||
       rot_dims > 256 || (rot_dims > 0 && freq == nullptr) || (q_norm == nullptr) != (k_norm == nullptr))
     return -2;
   if (pool != nullptr && (block_table == nullptr || req_of_token == nullptr || slots == nullptr || status == nullptr ||
-                          v_at < dk || v_at + dv > row || page_size <= 0))
+                          v_at < maps * dk || v_at + dv > row || page_size <= 0 || k == nullptr))
     return -2;
-  const int units = n_heads + n_kv + ((unit_values || pool != nullptr) ? n_kv : 0);
+  if (k == nullptr && unit_values) return -2;
+  const int units = (n_heads + (k != nullptr ? n_kv : 0)) * maps + ((unit_values || pool != nullptr) ? n_kv : 0);
   // a warp a (token, head) in a step of few tokens; with many tokens a block takes more of a token's heads
   const int want = (148 * 40 + n_tokens - 1) / n_tokens, most = units < 4 * 1024 ? (units + 3) / 4 : 1024;
   const int rows = want < most ? want : most;
   const rl::QkvCacheTarget c{pool, block_table, ldt, req_of_token, slots, v_at, row, page_size, max_pages, status};
   if (pool != nullptr && cache_dtype == RL_F32)
     rl::launch_pdl(rl::qkv_norm_rotate_kernel<float>, dim3(n_tokens, rows), 128, 0, stream, q, ldq, k, ldk, v, ldv, q_norm,
-                   k_norm, freq, positions, n_tokens, n_heads, n_kv, dk, dv, rot_dims, unit_values, unit_qk, eps, c);
+                   k_norm, freq, positions, n_tokens, n_heads, n_kv, maps, dk, dv, rot_dims, rot_mult, unit_values, unit_qk, eps, c);
   else
     rl::launch_pdl(rl::qkv_norm_rotate_kernel<__nv_bfloat16>, dim3(n_tokens, rows), 128, 0, stream, q, ldq, k, ldk, v, ldv,
-                   q_norm, k_norm, freq, positions, n_tokens, n_heads, n_kv, dk, dv, rot_dims, unit_values, unit_qk, eps, c);
+                   q_norm, k_norm, freq, positions, n_tokens, n_heads, n_kv, maps, dk, dv, rot_dims, rot_mult, unit_values,
+                   unit_qk, eps, c);
   RL_CHECK_LAUNCH();
   return 0;
 }

@@ -67,7 +67,7 @@ __global__ __launch_bounds__(BM_THREADS) void bias_attn_mma_kernel(const BiasAtt
   }
   for (int i = tid; i < BM_KEYS * LDQ; i += BM_THREADS) Ks[i] = __float2bfloat16_rn(0.f);
   for (int i = tid; i < DVP * LDV; i += BM_THREADS) Vt[i] = __float2bfloat16_rn(0.f);
-  int row_pos[2], row_head[2];
+  int row_pos[2], row_lo[2], row_head[2];
   float row_mul[2], row_slope[2], m[2], l[2];
   bool row_ok[2];
 #pragma unroll
@@ -75,6 +75,7 @@ __global__ __launch_bounds__(BM_THREADS) void bias_attn_mma_kernel(const BiasAtt
     const int r = warp * 16 + quad + 8 * a, tl = r / HB, hl = r - tl * HB;
     row_ok[a] = tl < n_tok && hb0 + hl < hg;
     row_pos[a] = pos0 + tl;
+    row_lo[a] = bias_first_seen(p, row_pos[a]);
     row_head[a] = g * hg + hb0 + hl;
     float temp = 1.0f;
     if (p.temp_every > 0) temp = 1.0f + p.temp_coef * logf((float)((row_pos[a] + 1) / p.temp_every + 1));
@@ -88,7 +89,7 @@ __global__ __launch_bounds__(BM_THREADS) void bias_attn_mma_kernel(const BiasAtt
 #pragma unroll
   for (int nt = 0; nt < DVT; ++nt) o[nt][0] = o[nt][1] = o[nt][2] = o[nt][3] = 0.f;
   const int last_pos = pos0 + n_tok - 1;
-  const int first_seen = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;  // the earliest key any row of the block sees
+  const int first_seen = bias_first_seen(p, pos0);  // the earliest key any row of the block sees
   const __nv_bfloat16* pool = reinterpret_cast<const __nv_bfloat16*>(p.pool);
   const int* table = p.block_table + (size_t)slot * p.ldt;
   auto locate = [&](int j0, int buf) {
@@ -177,7 +178,7 @@ __global__ __launch_bounds__(BM_THREADS) void bias_attn_mma_kernel(const BiasAtt
         for (int e = 0; e < 2; ++e) {
           const int j = j0 + nt * 8 + 2 * in_quad + e;
           float& v = s[nt][2 * a + e];
-          const bool see = row_ok[a] && j <= row_pos[a] && (p.window <= 0 || row_pos[a] - j < p.window);
+          const bool see = row_ok[a] && j <= row_pos[a] && j >= row_lo[a];
           v = see ? v * row_mul[a] - row_slope[a] * (float)(row_pos[a] - j) : -CUDART_INF_F;
           tile_max = fmaxf(tile_max, v);
         }
@@ -272,12 +273,19 @@ __device__ __forceinline__ void bm_ldmatrix_x4_trans(uint32_t (&r)[4], uint32_t 
                : "r"(addr));
 }
 
-template <int DKT, int DVT>
-__global__ __launch_bounds__(BM_THREADS, (DVT <= 8 ? 4 : 3)) void bias_attn_mma_async_kernel(const BiasAttnParams p) {
+//
+// With two maps a block has four more warps: warps 0-3 take the rows' map 1, warps 4-7 their map 2, over the same key
+// and value tiles (a key row in shared memory holds both keys, each filled up to DKP entries); at the end the second
+// map's results meet the first's through shared memory.
+template <int DKT, int DVT, int MAPS>
+__global__ __launch_bounds__(BM_THREADS * MAPS, (MAPS == 2 ? 2 : (DVT <= 8 ? 4 : 3)))
+void bias_attn_mma_async_kernel(const BiasAttnParams p) {
   extern __shared__ __align__(16) unsigned char bm_s[];
   pdl_begin();
+  constexpr int THREADS = BM_THREADS * MAPS;
   constexpr int DKP = 16 * DKT, DVP = 8 * DVT;
-  constexpr int LDQ = DKP + BM_PAD, LDW = DVP + BM_PAD;  // row strides in elements (multiples of 8: 16-byte rows)
+  // row strides in elements (multiples of 8: 16-byte rows)
+  constexpr int LDQ = DKP + BM_PAD, LDK = MAPS * DKP + BM_PAD, LDW = DVP + BM_PAD;
   const int subs = p.tile_tokens / p.tokens_per_block;
   // a portion's last tiles walk the most keys: taken first, they do not run alone at the end
   const int bx = gridDim.x - 1 - blockIdx.x;
@@ -292,24 +300,26 @@ __global__ __launch_bounds__(BM_THREADS, (DVT <= 8 ? 4 : 3)) void bias_attn_mma_
   const int g = blockIdx.y, hg = p.n_heads / p.n_kv;
   const int HB = p.heads_per_block, hb0 = blockIdx.z * HB;
   const int dk = p.dk, dv = p.dv;
-  __nv_bfloat16* Qs = reinterpret_cast<__nv_bfloat16*>(bm_s);  // [BM_ROWS][LDQ]
-  __nv_bfloat16* Kr = Qs + BM_ROWS * LDQ;                       // [2][BM_KEYS][LDQ]
-  __nv_bfloat16* Vr = Kr + 2 * BM_KEYS * LDQ;                   // [2][BM_KEYS][LDW]: row by row
+  __nv_bfloat16* Qs = reinterpret_cast<__nv_bfloat16*>(bm_s);  // [MAPS][BM_ROWS][LDQ]
+  __nv_bfloat16* Kr = Qs + MAPS * BM_ROWS * LDQ;                // [2][BM_KEYS][LDK]
+  __nv_bfloat16* Vr = Kr + 2 * BM_KEYS * LDK;                   // [2][BM_KEYS][LDW]: row by row
   __shared__ const __nv_bfloat16* key_src[2][BM_KEYS];
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int tid = threadIdx.x, map = MAPS == 2 ? tid / BM_THREADS : 0;
+  const int warp = (tid >> 5) - map * (BM_THREADS / 32), lane = tid & 31;  // the warp among those of its map
   const int quad = lane >> 2, in_quad = lane & 3;
-  for (int i = tid; i < BM_ROWS * DKP; i += BM_THREADS) {
-    const int r = i / DKP, d = i - r * DKP;
+  for (int i = tid; i < MAPS * BM_ROWS * DKP; i += THREADS) {
+    const int row = i / DKP, d = i - row * DKP;
+    const int qm = MAPS == 2 ? row / BM_ROWS : 0, r = row - qm * BM_ROWS;
     const int tl = r / HB, hl = r - tl * HB;
     float v = 0.f;
     if (tl < n_tok && hb0 + hl < hg && d < dk)
-      v = p.q[(size_t)(t_begin + first + tl) * p.ldq + (size_t)(g * hg + hb0 + hl) * dk + d];
-    Qs[r * LDQ + d] = __float2bfloat16_rn(v);
+      v = p.q[(size_t)(t_begin + first + tl) * p.ldq + ((size_t)(g * hg + hb0 + hl) * MAPS + qm) * dk + d];
+    Qs[row * LDQ + d] = __float2bfloat16_rn(v);
   }
   // entries beyond dk and dv are never copied: they stay zero
-  for (int i = tid; i < 2 * BM_KEYS * LDQ; i += BM_THREADS) Kr[i] = __float2bfloat16_rn(0.f);
-  for (int i = tid; i < 2 * BM_KEYS * LDW; i += BM_THREADS) Vr[i] = __float2bfloat16_rn(0.f);
-  int row_pos[2], row_head[2];
+  for (int i = tid; i < 2 * BM_KEYS * LDK; i += THREADS) Kr[i] = __float2bfloat16_rn(0.f);
+  for (int i = tid; i < 2 * BM_KEYS * LDW; i += THREADS) Vr[i] = __float2bfloat16_rn(0.f);
+  int row_pos[2], row_lo[2], row_head[2];
   float row_mul[2], row_slope[2], m[2], l[2];
   bool row_ok[2];
 #pragma unroll
@@ -317,6 +327,7 @@ __global__ __launch_bounds__(BM_THREADS, (DVT <= 8 ? 4 : 3)) void bias_attn_mma_
     const int r = warp * 16 + quad + 8 * a, tl = r / HB, hl = r - tl * HB;
     row_ok[a] = tl < n_tok && hb0 + hl < hg;
     row_pos[a] = pos0 + tl;
+    row_lo[a] = bias_first_seen(p, row_pos[a]);
     row_head[a] = g * hg + hb0 + hl;
     float temp = 1.0f;
     if (p.temp_every > 0) temp = 1.0f + p.temp_coef * logf((float)((row_pos[a] + 1) / p.temp_every + 1));
@@ -330,7 +341,7 @@ __global__ __launch_bounds__(BM_THREADS, (DVT <= 8 ? 4 : 3)) void bias_attn_mma_
 #pragma unroll
   for (int nt = 0; nt < DVT; ++nt) o[nt][0] = o[nt][1] = o[nt][2] = o[nt][3] = 0.f;
   const int last_pos = pos0 + n_tok - 1;
-  const int first_seen = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;
+  const int first_seen = bias_first_seen(p, pos0), last_lo = bias_first_seen(p, last_pos);
   const __nv_bfloat16* pool = reinterpret_cast<const __nv_bfloat16*>(p.pool);
   const int* table = p.block_table + (size_t)slot * p.ldt;
   auto locate = [&](int j0, int buf) {
@@ -348,17 +359,18 @@ __global__ __launch_bounds__(BM_THREADS, (DVT <= 8 ? 4 : 3)) void bias_attn_mma_
       key_src[buf][tid] = src;
     }
   };
-  const int kp = dk / 8, vp = dv / 8, per_key = kp + vp;
+  const int k1 = dk / 8, kp = MAPS * k1, vp = dv / 8, per_key = kp + vp;
   // the copies of one tile into stage `st`, from the places in key_src[st]; keys nobody sees get zeros
   auto fetch = [&](int st) {
-    __nv_bfloat16* kd = Kr + st * BM_KEYS * LDQ;
+    __nv_bfloat16* kd = Kr + st * BM_KEYS * LDK;
     __nv_bfloat16* vd = Vr + st * BM_KEYS * LDW;
-    for (int i = tid; i < BM_KEYS * per_key; i += BM_THREADS) {
+    for (int i = tid; i < BM_KEYS * per_key; i += THREADS) {
       const int jj = i / per_key, piece = i - jj * per_key;
       const __nv_bfloat16* src = key_src[st][jj];
       const bool is_v = piece >= kp;
       const int at = is_v ? (piece - kp) * 8 : piece * 8;
-      __nv_bfloat16* dst = is_v ? vd + jj * LDW + at : kd + jj * LDQ + at;
+      const int k_at = MAPS == 2 && piece >= k1 ? DKP + at - dk : at;  // the second key's place in the tile's row
+      __nv_bfloat16* dst = is_v ? vd + jj * LDW + at : kd + jj * LDK + k_at;
       if (src != nullptr) bm_cp_async16((uint32_t)__cvta_generic_to_shared(dst), src + (is_v ? p.v_at : 0) + at);
       else *reinterpret_cast<uint4*>(dst) = make_uint4(0u, 0u, 0u, 0u);
     }
@@ -373,13 +385,13 @@ __global__ __launch_bounds__(BM_THREADS, (DVT <= 8 ? 4 : 3)) void bias_attn_mma_
   __syncthreads();  // every thread has read the first tile's places
   locate(j_begin + 2 * BM_KEYS, 0);
   // the queries' fragments do not change from tile to tile: in registers once, where the key size leaves room
-  constexpr bool Q_IN_REGS = DKT <= 4;
+  constexpr bool Q_IN_REGS = DKT <= 4 && (MAPS == 1 || DVT <= 8);
   const uint32_t* Qw = reinterpret_cast<const uint32_t*>(Qs);
   uint32_t qa[Q_IN_REGS ? DKT : 1][4];
   if (Q_IN_REGS) {
 #pragma unroll
     for (int kc = 0; kc < DKT; ++kc) {
-      const int qrow = warp * 16 + quad, qw = kc * 8 + in_quad;  // in 32-bit words
+      const int qrow = map * BM_ROWS + warp * 16 + quad, qw = kc * 8 + in_quad;  // in 32-bit words
       qa[kc][0] = Qw[qrow * (LDQ / 2) + qw];
       qa[kc][1] = Qw[(qrow + 8) * (LDQ / 2) + qw];
       qa[kc][2] = Qw[qrow * (LDQ / 2) + qw + 4];
@@ -398,7 +410,7 @@ __global__ __launch_bounds__(BM_THREADS, (DVT <= 8 ? 4 : 3)) void bias_attn_mma_
     }
     __syncthreads();  // this tile has arrived for every thread; the next tile's places have been read
     if (more) locate(j0 + 3 * BM_KEYS, st ^ 1);
-    const __nv_bfloat16* Ks = Kr + st * BM_KEYS * LDQ;
+    const __nv_bfloat16* Ks = Kr + st * BM_KEYS * LDK + map * DKP;
     const __nv_bfloat16* Vs = Vr + st * BM_KEYS * LDW;
     float s[BM_KEYS / 8][4];
 #pragma unroll
@@ -411,7 +423,7 @@ __global__ __launch_bounds__(BM_THREADS, (DVT <= 8 ? 4 : 3)) void bias_attn_mma_
       if (Q_IN_REGS) {
         a[0] = qa[kc][0], a[1] = qa[kc][1], a[2] = qa[kc][2], a[3] = qa[kc][3];
       } else {
-        const int qrow = warp * 16 + quad, qw = kc * 8 + in_quad;  // in 32-bit words
+        const int qrow = map * BM_ROWS + warp * 16 + quad, qw = kc * 8 + in_quad;  // in 32-bit words
         a[0] = Qw[qrow * (LDQ / 2) + qw];
         a[1] = Qw[(qrow + 8) * (LDQ / 2) + qw];
         a[2] = Qw[qrow * (LDQ / 2) + qw + 4];
@@ -421,15 +433,15 @@ __global__ __launch_bounds__(BM_THREADS, (DVT <= 8 ? 4 : 3)) void bias_attn_mma_
       for (int nt = 0; nt < BM_KEYS / 8; nt += 2) {
         uint32_t kf[4];
         const int key = (nt + (lane >> 4)) * 8 + (lane & 7);
-        bm_ldmatrix_x4(kf, (uint32_t)__cvta_generic_to_shared(Ks + key * LDQ + kc * 16 + ((lane >> 3) & 1) * 8));
+        bm_ldmatrix_x4(kf, (uint32_t)__cvta_generic_to_shared(Ks + key * LDK + kc * 16 + ((lane >> 3) & 1) * 8));
         mma_bf16_16816(s[nt], a, kf[0], kf[1]);
         mma_bf16_16816(s[nt + 1], a, kf[2], kf[3]);
       }
     }
     uint32_t pa[BM_KEYS / 16][4];
     // a tile that every row of the block sees whole (all of it at or before the block's first position and
-    // inside the last row's window) needs no mask
-    const bool whole = j0 + BM_KEYS - 1 <= pos0 && (p.window <= 0 || last_pos - j0 < p.window);
+    // inside the last row's window or chunk) needs no mask
+    const bool whole = j0 + BM_KEYS - 1 <= pos0 && j0 >= last_lo;
 #pragma unroll
     for (int a = 0; a < 2; ++a) {
       float tile_max = -CUDART_INF_F;
@@ -450,7 +462,7 @@ __global__ __launch_bounds__(BM_THREADS, (DVT <= 8 ? 4 : 3)) void bias_attn_mma_
           for (int e = 0; e < 2; ++e) {
             const int j = j0 + nt * 8 + 2 * in_quad + e;
             float& v = s[nt][2 * a + e];
-            const bool see = row_ok[a] && j <= row_pos[a] && (p.window <= 0 || row_pos[a] - j < p.window);
+            const bool see = row_ok[a] && j <= row_pos[a] && j >= row_lo[a];
             v = see ? v * row_mul[a] - row_slope[a] * (float)(row_pos[a] - j) : -CUDART_INF_F;
             tile_max = fmaxf(tile_max, v);
           }
@@ -505,47 +517,99 @@ __global__ __launch_bounds__(BM_THREADS, (DVT <= 8 ? 4 : 3)) void bias_attn_mma_
       }
     }
   }
+  if constexpr (MAPS == 2) {
+    constexpr int LDO = DVP + 2;  // a quad's lanes write neighbouring pairs of columns, quads neighbouring rows
+    float* second = reinterpret_cast<float*>(bm_s);  // [BM_ROWS][LDO]: queries, keys and values have been used
+    static_assert((size_t)BM_ROWS * LDO * 4 <= ((size_t)2 * BM_ROWS * LDQ + 2 * BM_KEYS * LDK + 2 * BM_KEYS * LDW) * 2, "fits");
+    __syncthreads();
+    if (map == 1) {
 #pragma unroll
-  for (int a = 0; a < 2; ++a) {
-    if (!row_ok[a]) continue;
-    const int r = warp * 16 + quad + 8 * a;
-    const int tok = t_begin + first + r / HB;
-    const float inv = 1.0f / (l[a] + (p.sink != nullptr ? expf(p.sink[row_head[a]] - m[a]) : 0.f));
-    __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)tok * p.ldo + (size_t)row_head[a] * dv;
-    int gs;
-    const float* gr = bias_gate_row(p, tok, row_head[a], gs);
+      for (int a = 0; a < 2; ++a) {
+        const float inv = row_ok[a] ? 1.0f / l[a] : 0.f;
+        float* to = second + (warp * 16 + quad + 8 * a) * LDO + 2 * in_quad;
 #pragma unroll
-    for (int nt = 0; nt < DVT; ++nt) {
+        for (int nt = 0; nt < DVT; ++nt) *reinterpret_cast<float2*>(to + nt * 8) = make_float2(o[nt][2 * a] * inv, o[nt][2 * a + 1] * inv);
+      }
+    }
+    __syncthreads();
+    if (map == 1) return;
+    const float lambda = *p.diff_lambda;
 #pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const int col = nt * 8 + 2 * in_quad + e;
-        if (col < dv) {
-          float v = o[nt][2 * a + e] * inv;
-          if (gr != nullptr) v *= 1.0f / (1.0f + expf(-gr[col * gs]));
-          out[col] = __float2bfloat16_rn(v);
+    for (int a = 0; a < 2; ++a) {
+      const int r = warp * 16 + quad + 8 * a;
+      const float inv = row_ok[a] ? 1.0f / l[a] : 0.f;
+      const float* from = second + r * LDO + 2 * in_quad;
+      float ss = 0.f;
+#pragma unroll
+      for (int nt = 0; nt < DVT; ++nt) {  // columns beyond dv are zero in both maps
+        const float2 b = *reinterpret_cast<const float2*>(from + nt * 8);
+        o[nt][2 * a] = fmaf(-lambda, b.x, o[nt][2 * a] * inv);
+        o[nt][2 * a + 1] = fmaf(-lambda, b.y, o[nt][2 * a + 1] * inv);
+        ss = fmaf(o[nt][2 * a], o[nt][2 * a], fmaf(o[nt][2 * a + 1], o[nt][2 * a + 1], ss));
+      }
+      ss += __shfl_xor_sync(0xffffffffu, ss, 1);
+      ss += __shfl_xor_sync(0xffffffffu, ss, 2);
+      const float mul = p.diff_mul / sqrtf(ss / (float)dv + p.diff_eps);
+      if (!row_ok[a]) continue;
+      __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)(t_begin + first + r / HB) * p.ldo + (size_t)row_head[a] * dv;
+#pragma unroll
+      for (int nt = 0; nt < DVT; ++nt)
+#pragma unroll
+        for (int e = 0; e < 2; ++e)
+          if (nt * 8 + 2 * in_quad + e < dv) out[nt * 8 + 2 * in_quad + e] = __float2bfloat16_rn(o[nt][2 * a + e] * mul);
+    }
+  } else {
+#pragma unroll
+    for (int a = 0; a < 2; ++a) {
+      if (!row_ok[a]) continue;
+      const int r = warp * 16 + quad + 8 * a;
+      const int tok = t_begin + first + r / HB;
+      const float inv = 1.0f / (l[a] + (p.sink != nullptr ? expf(p.sink[row_head[a]] - m[a]) : 0.f));
+      __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)tok * p.ldo + (size_t)row_head[a] * dv;
+      int gs;
+      const float* gr = bias_gate_row(p, tok, row_head[a], gs);
+#pragma unroll
+      for (int nt = 0; nt < DVT; ++nt) {
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const int col = nt * 8 + 2 * in_quad + e;
+          if (col < dv) {
+            float v = o[nt][2 * a + e] * inv;
+            if (gr != nullptr) v *= 1.0f / (1.0f + expf(-gr[col * gs]));
+            out[col] = __float2bfloat16_rn(v);
+          }
         }
       }
     }
   }
 }
 
+template <int DKT, int DVT, int MAPS>
+static void launch_bias_attn_mma_async(const BiasAttnParams& p, dim3 grid, cudaStream_t stream) {
+  constexpr int LDQA = 16 * DKT + BM_PAD, LDKA = MAPS * 16 * DKT + BM_PAD, LDWA = 8 * DVT + BM_PAD;
+  const size_t smem = ((size_t)MAPS * BM_ROWS * LDQA + (size_t)2 * BM_KEYS * LDKA + (size_t)2 * BM_KEYS * LDWA) * sizeof(__nv_bfloat16);
+  auto kernel = bias_attn_mma_async_kernel<DKT, DVT, MAPS>;
+  // all of an SM's memory as shared memory, so that as many of its larger blocks fit as registers allow
+  static bool raised = false;
+  if (!raised) {
+    note_launch(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024));
+    note_launch(cudaFuncSetAttribute(kernel, cudaFuncAttributePreferredSharedMemoryCarveout,
+                                     (int)cudaSharedmemCarveoutMaxShared));
+    raised = true;
+  }
+  launch_pdl_split(false, kernel, grid, BM_THREADS * MAPS, smem, stream, p);
+}
+
 template <int DKT, int DVT>
-static void launch_bias_attn_mma(const BiasAttnParams& p, dim3 grid, cudaStream_t stream) {
-  // cache rows in 16-byte pieces: the form whose tiles travel by cp.async (all of an SM's memory as shared memory,
-  // so that as many of its larger blocks fit as registers allow)
+static void launch_bias_attn_mma(const BiasAttnParams& p, int maps, dim3 grid, cudaStream_t stream) {
+  // cache rows in 16-byte pieces: the form whose tiles travel by cp.async (two maps: the only one)
+  if (maps == 2) {
+    launch_bias_attn_mma_async<DKT, DVT, 2>(p, grid, stream);
+    return;
+  }
   if (BIAS_ATTENTION_ASYNC && p.dk % 8 == 0 && p.dv % 8 == 0 && p.v_at % 8 == 0 && p.row % 8 == 0 &&
       (reinterpret_cast<uintptr_t>(p.pool) & 15) == 0) {
-    constexpr int LDQA = 16 * DKT + BM_PAD, LDWA = 8 * DVT + BM_PAD;
-    const size_t smem_a = ((size_t)BM_ROWS * LDQA + (size_t)2 * BM_KEYS * LDQA + (size_t)2 * BM_KEYS * LDWA) * sizeof(__nv_bfloat16);
-    auto kernel_a = bias_attn_mma_async_kernel<DKT, DVT>;
-    static bool raised_a = false;
-    if (!raised_a) {
-      note_launch(cudaFuncSetAttribute(kernel_a, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024));
-      note_launch(cudaFuncSetAttribute(kernel_a, cudaFuncAttributePreferredSharedMemoryCarveout,
-                                       (int)cudaSharedmemCarveoutMaxShared));
-      raised_a = true;
-    }
-    launch_pdl_split(false, kernel_a, grid, BM_THREADS, smem_a, stream, p);
+    launch_bias_attn_mma_async<DKT, DVT, 1>(p, grid, stream);
     return;
   }
   constexpr int LDQ = 16 * DKT + BM_PAD, LDV = BM_KEYS + BM_PAD;
@@ -562,18 +626,18 @@ static void launch_bias_attn_mma(const BiasAttnParams& p, dim3 grid, cudaStream_
 }
 
 // dk, dv <= 128
-static void dispatch_bias_attn_mma(const BiasAttnParams& p, dim3 grid, cudaStream_t stream) {
+static void dispatch_bias_attn_mma(const BiasAttnParams& p, int maps, dim3 grid, cudaStream_t stream) {
   const int kt = p.dk <= 32 ? 0 : (p.dk <= 64 ? 1 : 2), vt = p.dv <= 32 ? 0 : (p.dv <= 64 ? 1 : 2);
   switch (kt * 3 + vt) {
-    case 0: launch_bias_attn_mma<2, 4>(p, grid, stream); break;
-    case 1: launch_bias_attn_mma<2, 8>(p, grid, stream); break;
-    case 2: launch_bias_attn_mma<2, 16>(p, grid, stream); break;
-    case 3: launch_bias_attn_mma<4, 4>(p, grid, stream); break;
-    case 4: launch_bias_attn_mma<4, 8>(p, grid, stream); break;
-    case 5: launch_bias_attn_mma<4, 16>(p, grid, stream); break;
-    case 6: launch_bias_attn_mma<8, 4>(p, grid, stream); break;
-    case 7: launch_bias_attn_mma<8, 8>(p, grid, stream); break;
-    default: launch_bias_attn_mma<8, 16>(p, grid, stream); break;
+    case 0: launch_bias_attn_mma<2, 4>(p, maps, grid, stream); break;
+    case 1: launch_bias_attn_mma<2, 8>(p, maps, grid, stream); break;
+    case 2: launch_bias_attn_mma<2, 16>(p, maps, grid, stream); break;
+    case 3: launch_bias_attn_mma<4, 4>(p, maps, grid, stream); break;
+    case 4: launch_bias_attn_mma<4, 8>(p, maps, grid, stream); break;
+    case 5: launch_bias_attn_mma<4, 16>(p, maps, grid, stream); break;
+    case 6: launch_bias_attn_mma<8, 4>(p, maps, grid, stream); break;
+    case 7: launch_bias_attn_mma<8, 8>(p, maps, grid, stream); break;
+    default: launch_bias_attn_mma<8, 16>(p, maps, grid, stream); break;
   }
 }
 

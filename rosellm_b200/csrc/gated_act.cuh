@@ -1,5 +1,6 @@
 // Gated activations of feed-forward layers with two input projections, gate g and up u:
-// the unit's value is f(g, u).  Arithmetic in float32.
+// the unit's value is f(g, u); and activations of layers with one input projection, f(u).
+// Arithmetic in float32.
 #pragma once
 #include "common.cuh"
 
@@ -7,6 +8,9 @@
 #define RL_GATE_SILU 1           // g * sigmoid(g) * u
 #define RL_GATE_GELU_TANH 2      // gelu_tanh(g) * u
 #define RL_GATE_CLAMPED_SWISH 3  // g' = min(g, limit), u' = clamp(u, -limit, limit): g' * sigmoid(alpha g') * (u' + 1)
+#define RL_UNIT_RELU_SQUARED 4   // one projection: max(u, 0)^2
+#define RL_UNIT_FIRST 4          // kinds from here on take one projection
+#define RL_UNIT_LAST 4
 
 namespace rl {
 
@@ -26,6 +30,12 @@ __device__ __forceinline__ float gated_value(float g, float u, int kind, float a
       return g / (1.0f + expf(-alpha * g)) * (u + 1.0f);
     }
   }
+}
+
+// f(u) of a layer with one input projection.  One kind so far, so nothing to choose.
+__device__ __forceinline__ float unit_value(float u, int /*kind*/) {
+  const float r = fmaxf(u, 0.f);
+  return r * r;
 }
 
 }  // namespace rl

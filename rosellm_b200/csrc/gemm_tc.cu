@@ -418,6 +418,9 @@ __global__ __launch_bounds__(PTHREADS, 1) void gemm_tc_persistent_kernel(const _
         } else if (p.act == RL_ACT_GELU_ERF) {
 #pragma unroll
           for (int i = 0; i < 32; ++i) v[i] = act_fn(v[i] + __shfl_sync(0xffffffffu, bias_c, i), RL_ACT_GELU_ERF);
+        } else if (p.act == RL_ACT_RELU_SQUARED) {
+#pragma unroll
+          for (int i = 0; i < 32; ++i) v[i] = act_fn(v[i] + __shfl_sync(0xffffffffu, bias_c, i), RL_ACT_RELU_SQUARED);
         } else {
 #pragma unroll
           for (int i = 0; i < 32; ++i) v[i] += __shfl_sync(0xffffffffu, bias_c, i);

@@ -1,8 +1,8 @@
 // Mixture of experts: routing, and the experts' gated feed-forward as grouped products.
 //
 // Routing (`moe_select_kernel`, one warp per token, float32): scores s = softmax(z) over all
-// experts, or (score_kind 1) s = sigmoid(z) of each expert by itself; the choice is made on s + correction,
-// the weights are the chosen experts' s.  With
+// experts, or (score_kind 1) s = sigmoid(z) of each expert by itself, or (score_kind 2) s = z; the choice is made on
+// s + correction, the weights are the chosen experts' s, with score_kind 2 the softmax over the chosen s alone.  With
 // groups, the experts form `group_count` equal groups of neighbours, a group's score is the
 // largest choice score in it, and only experts of the best `group_keep` groups can be chosen
 // (the others count as minus infinity).  Ties go to the lower index.
@@ -17,6 +17,9 @@
 // weight belongs on the expert's INPUT instead (expert(w * h)), `moe_scatter_kernel` leaves each
 // place's weight in `place_weight`, the first product scales its two results by it before the
 // gate function (W (w h) = w (W h)), and the sum at the end takes no weights.
+// Experts may also have one input projection instead of two (kinds from RL_UNIT_FIRST on): f(h W_up^T).
+// `moe_combine_kernel` also adds the output of a feed-forward that every token passes beside its experts, times a
+// sigmoid of one logit a token, where the caller gives it.
 // Products: float32 as IEEE multiply-adds on 64 x 64 tiles (tile_gemm.cuh); bfloat16 on the tensor
 // cores (mma_tile.cuh) with float32 accumulation, or, where an expert has a few rows only (decode
 // steps), by `moe_rows_kernel`, which streams the weights once with a warp an output column.
@@ -31,6 +34,7 @@ namespace rl {
 
 constexpr int MOE_TILE_ROWS = TG_M;
 constexpr float MOE_TAKEN = 1e38f;  // marks a group that has been picked
+constexpr int MOE_SCORE_SOFTMAX = 0, MOE_SCORE_SIGMOID = 1, MOE_SCORE_CHOSEN_SOFTMAX = 2;
 
 // The lane's candidate (value, index) merged over the warp: the largest value, among equals the
 // lowest index.
@@ -46,24 +50,61 @@ __device__ __forceinline__ void warp_argmax(float& v, int& idx) {
   }
 }
 
-__global__ __launch_bounds__(128) void moe_select_kernel(const float* __restrict__ z, long ldz,
-                                                         const float* __restrict__ correction, int n_tokens,
-                                                         int n_experts, int top, int group_count, int group_keep,
-                                                         int score_kind, int* __restrict__ ids, float* __restrict__ weights,
-                                                         int* __restrict__ counts) {
-  extern __shared__ float smem[];
-  pdl_begin();
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const int t = blockIdx.x * 4 + warp;
-  if (t >= n_tokens) return;
-  const int E = n_experts;
-  float* s_w = smem + (size_t)warp * 3 * E;  // scores
-  float* c_w = s_w + E;                      // choice scores
-  float* g_w = c_w + E;                      // group scores
-  const float* zr = z + (size_t)t * ldz;
+// What a block with the pairs' counts in shared memory does to lay them out expert by expert: offsets, tile list and a
+// place for every pair (`ids` as this block wrote them, a barrier before).  count_s is used up; off_s and tile_s are
+// scratch of E + 1 entries.
+constexpr int MOE_ROUTE_MAX_PAIRS = 8192, MOE_ROUTE_MAX_EXPERTS = 2048;
+
+__device__ __forceinline__ void moe_layout_block(int n_pairs, int top, int n_experts, int* count_s, int* off_s, int* tile_s,
+                                                 const int* ids, int* offsets, int* tiles, int* meta, int* row_token,
+                                                 int* place_of, const float* weights, float* place_weight) {
+  if (threadIdx.x == 0) {
+    int at = 0, tile = 0;
+    for (int e = 0; e < n_experts; ++e) {
+      off_s[e] = at;
+      tile_s[e] = tile;
+      at += count_s[e];
+      tile += (count_s[e] + MOE_TILE_ROWS - 1) / MOE_TILE_ROWS;
+    }
+    off_s[n_experts] = at;
+    tile_s[n_experts] = tile;
+    meta[0] = tile;
+  }
+  __syncthreads();
+  for (int e = threadIdx.x; e < n_experts; e += blockDim.x) {
+    const int c = off_s[e + 1] - off_s[e];
+    for (int k = 0; k * MOE_TILE_ROWS < c; ++k) {
+      int* tl = tiles + 3 * (size_t)(tile_s[e] + k);
+      tl[0] = e;
+      tl[1] = off_s[e] + k * MOE_TILE_ROWS;
+      tl[2] = min(MOE_TILE_ROWS, c - k * MOE_TILE_ROWS);
+    }
+    offsets[e] = off_s[e];
+    count_s[e] = 0;  // from here on: the places handed out
+  }
+  if (threadIdx.x == 0) offsets[n_experts] = off_s[n_experts];
+  __syncthreads();
+  for (int i = threadIdx.x; i < n_pairs; i += blockDim.x) {
+    const int e = ids[i];
+    const int place = off_s[e] + atomicAdd(&count_s[e], 1);
+    row_token[place] = i / top;
+    place_of[i] = place;
+    if (place_weight != nullptr) place_weight[place] = weights[i];
+  }
+}
+
+// Routing of one token by one warp: the `top` experts of router logits zr[E] into ids_t / weights_t, and one more pair
+// counted for each.  s_w, c_w, g_w: the warp's scratch in shared memory, E floats each (scores, choice scores, group
+// scores).
+__device__ __forceinline__ void moe_select_token(const float* __restrict__ zr, const float* __restrict__ correction, int E,
+                                                 int top, int group_count, int group_keep, int score_kind, float* s_w,
+                                                 float* c_w, float* g_w, int* ids_t, float* weights_t, int* counts,
+                                                 int lane) {
   float sum = 1.f;
-  if (score_kind == 1) {
+  if (score_kind == MOE_SCORE_SIGMOID) {
     for (int e = lane; e < E; e += 32) s_w[e] = 1.0f / (1.0f + expf(-zr[e]));
+  } else if (score_kind == MOE_SCORE_CHOSEN_SOFTMAX) {
+    for (int e = lane; e < E; e += 32) s_w[e] = zr[e];
   } else {
     float mx = -CUDART_INF_F;
     for (int e = lane; e < E; e += 32) mx = fmaxf(mx, zr[e]);
@@ -77,7 +118,7 @@ __global__ __launch_bounds__(128) void moe_select_kernel(const float* __restrict
     sum = warp_sum(sum);
   }
   for (int e = lane; e < E; e += 32) {
-    const float s = score_kind == 1 ? s_w[e] : s_w[e] / sum;
+    const float s = score_kind == MOE_SCORE_SOFTMAX ? s_w[e] / sum : s_w[e];
     s_w[e] = s;
     c_w[e] = s + (correction != nullptr ? correction[e] : 0.f);
   }
@@ -121,13 +162,69 @@ __global__ __launch_bounds__(128) void moe_select_kernel(const float* __restrict
     warp_argmax(v, idx);
     if (idx == 0x7fffffff) idx = 0;  // fewer allowed experts than `top`: refused by the host before
     if (lane == 0) {
-      ids[(size_t)t * top + j] = idx;
-      weights[(size_t)t * top + j] = s_w[idx];
+      ids_t[j] = idx;
+      weights_t[j] = s_w[idx];
+      g_w[j] = s_w[idx];  // the groups have been used
       atomicAdd(&counts[idx], 1);
       c_w[idx] = -CUDART_INF_F;
     }
     __syncwarp();
   }
+  if (score_kind == MOE_SCORE_CHOSEN_SOFTMAX) {  // the weights: a softmax over the chosen experts' logits alone
+    float mx = -CUDART_INF_F;
+    for (int j = lane; j < top; j += 32) mx = fmaxf(mx, g_w[j]);
+    mx = warp_max(mx);
+    float total = 0.f;
+    for (int j = lane; j < top; j += 32) total += expf(g_w[j] - mx);
+    total = warp_sum(total);
+    for (int j = lane; j < top; j += 32) weights_t[j] = expf(g_w[j] - mx) / total;
+    __syncwarp();
+  }
+}
+
+__global__ __launch_bounds__(128) void moe_select_kernel(const float* __restrict__ z, long ldz,
+                                                         const float* __restrict__ correction, int n_tokens,
+                                                         int n_experts, int top, int group_count, int group_keep,
+                                                         int score_kind, int* __restrict__ ids, float* __restrict__ weights,
+                                                         int* __restrict__ counts) {
+  extern __shared__ float smem[];
+  pdl_begin();
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int t = blockIdx.x * 4 + warp;
+  if (t >= n_tokens) return;
+  float* s_w = smem + (size_t)warp * 3 * n_experts;
+  moe_select_token(z + (size_t)t * ldz, correction, n_experts, top, group_count, group_keep, score_kind, s_w,
+                   s_w + n_experts, s_w + 2 * n_experts, ids + (size_t)t * top, weights + (size_t)t * top, counts, lane);
+}
+
+// The same routing with its layout, in one block (fused: choice, counts, offsets, tile list and places, which a decode
+// step would otherwise spend three launches on).  Each of the block's warps routes tokens in turn; counts live in
+// shared memory.  Dynamic shared memory: 3 E floats a warp.
+constexpr int MOE_ROUTE_MAX_TOKENS = 128;
+
+__global__ __launch_bounds__(1024, 1) void moe_select_route_kernel(const float* __restrict__ z, long ldz,
+                                                                const float* __restrict__ correction, int n_tokens,
+                                                                int n_experts, int top, int group_count, int group_keep,
+                                                                int score_kind, int* __restrict__ ids,
+                                                                float* __restrict__ weights, int* __restrict__ offsets,
+                                                                int* __restrict__ tiles, int* __restrict__ meta,
+                                                                int* __restrict__ row_token, int* __restrict__ place_of,
+                                                                float* __restrict__ place_weight) {
+  extern __shared__ float smem[];
+  __shared__ int count_s[MOE_ROUTE_MAX_EXPERTS], off_s[MOE_ROUTE_MAX_EXPERTS + 1], tile_s[MOE_ROUTE_MAX_EXPERTS + 1];
+  pdl_begin();
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5;
+  for (int e = threadIdx.x; e < n_experts; e += blockDim.x) count_s[e] = 0;
+  __syncthreads();
+  float* s_w = smem + (size_t)warp * 3 * n_experts;
+  for (int t = warp; t < n_tokens; t += n_warps) {
+    moe_select_token(z + (size_t)t * ldz, correction, n_experts, top, group_count, group_keep, score_kind, s_w,
+                     s_w + n_experts, s_w + 2 * n_experts, ids + (size_t)t * top, weights + (size_t)t * top, count_s, lane);
+    __syncwarp();
+  }
+  __syncthreads();
+  moe_layout_block(n_tokens * top, top, n_experts, count_s, off_s, tile_s, ids, offsets, tiles, meta, row_token, place_of,
+                   weights, place_weight);
 }
 
 // Routing without a router: row `token id` of an integer table [vocab, top] names the token's experts (the entries
@@ -163,8 +260,6 @@ __global__ __launch_bounds__(256) void moe_table_select_kernel(const int* __rest
 // The same routing with its layout, in one block (fused: choice, counts, offsets, tile list and places, which a
 // step of few tokens would otherwise spend three launches on): the counts live in shared memory, the global
 // counters are not touched.  At most MOE_ROUTE_MAX_PAIRS pairs.
-constexpr int MOE_ROUTE_MAX_PAIRS = 8192, MOE_ROUTE_MAX_EXPERTS = 2048;
-
 __global__ __launch_bounds__(1024) void moe_table_route_kernel(const int* __restrict__ token_ids,
                                                                const int* __restrict__ table, int vocab, int n_tokens,
                                                                int n_experts, int top, float weight, int* __restrict__ ids,
@@ -197,38 +292,8 @@ __global__ __launch_bounds__(1024) void moe_table_route_kernel(const int* __rest
     atomicAdd(&count_s[e], 1);
   }
   __syncthreads();
-  if (threadIdx.x == 0) {
-    int at = 0, tile = 0;
-    for (int e = 0; e < n_experts; ++e) {
-      off_s[e] = at;
-      tile_s[e] = tile;
-      at += count_s[e];
-      tile += (count_s[e] + MOE_TILE_ROWS - 1) / MOE_TILE_ROWS;
-    }
-    off_s[n_experts] = at;
-    tile_s[n_experts] = tile;
-    meta[0] = tile;
-  }
-  __syncthreads();
-  for (int e = threadIdx.x; e < n_experts; e += blockDim.x) {
-    const int c = off_s[e + 1] - off_s[e];
-    for (int k = 0; k * MOE_TILE_ROWS < c; ++k) {
-      int* tl = tiles + 3 * (size_t)(tile_s[e] + k);
-      tl[0] = e;
-      tl[1] = off_s[e] + k * MOE_TILE_ROWS;
-      tl[2] = min(MOE_TILE_ROWS, c - k * MOE_TILE_ROWS);
-    }
-    offsets[e] = off_s[e];
-    count_s[e] = 0;  // from here on: the places handed out
-  }
-  if (threadIdx.x == 0) offsets[n_experts] = off_s[n_experts];
-  __syncthreads();
-  for (int i = threadIdx.x; i < n_pairs; i += blockDim.x) {
-    const int e = ids[i];  // this thread's own write
-    const int place = off_s[e] + atomicAdd(&count_s[e], 1);
-    row_token[place] = i / top;
-    place_of[i] = place;
-  }
+  moe_layout_block(n_pairs, top, n_experts, count_s, off_s, tile_s, ids, offsets, tiles, meta, row_token, place_of, nullptr,
+                   nullptr);
 }
 
 // One block.  offsets[e]: first place of expert e; tiles[k] = (expert, first place, rows);
@@ -284,8 +349,9 @@ __global__ void moe_scatter_kernel(const int* __restrict__ ids, const int* __res
   if (place_weight != nullptr) place_weight[place] = weights[i];
 }
 
-// act[place, f] = f(h[token] . W_gate[e, f], h[token] . W_up[e, f]).  w_gu: [experts][2][ff][hidden].
-template <typename T>
+// act[place, f] = f(h[token] . W_gate[e, f], h[token] . W_up[e, f]).  w_gu: [experts][2][ff][hidden]; without PAIR
+// f(h[token] . W_up[e, f]), w_gu: [experts][ff][hidden].
+template <typename T, bool PAIR>
 __global__ __launch_bounds__(256) void moe_ffn1_kernel(const T* __restrict__ h, long ldh, const T* __restrict__ w_gu,
                                                        const int* __restrict__ tiles, const int* __restrict__ meta,
                                                        const int* __restrict__ row_token,
@@ -293,7 +359,7 @@ __global__ __launch_bounds__(256) void moe_ffn1_kernel(const T* __restrict__ h, 
                                                        long lda, int hidden, int ff, int kind, float alpha,
                                                        float limit) {
   __shared__ TileGemmSmem s;
-  __shared__ float up_s[TG_K][TG_N + 1];
+  __shared__ float up_s[PAIR ? TG_K : 1][TG_N + 1];
   __shared__ int tok[TG_M];
   pdl_begin();
   if ((int)blockIdx.x >= meta[0]) return;
@@ -301,15 +367,18 @@ __global__ __launch_bounds__(256) void moe_ffn1_kernel(const T* __restrict__ h, 
   const int n0 = blockIdx.y * TG_N;
   if (threadIdx.x < TG_M) tok[threadIdx.x] = threadIdx.x < rows ? row_token[row0 + threadIdx.x] : 0;
   __syncthreads();
-  const T* wg = w_gu + (size_t)e * 2 * ff * hidden;
-  const T* wu = wg + (size_t)ff * hidden;
+  const T* wg = w_gu + (size_t)e * (PAIR ? 2 : 1) * ff * hidden;
+  const T* wu = wg + (PAIR ? (size_t)ff * hidden : 0);
   float acc_g[4][4] = {}, acc_u[4][4] = {};
-  tile_gemm_pair(
-      acc_g, acc_u, hidden,
-      [&](int m, int k) { return (m < rows && k < hidden) ? to_f32(h[(size_t)tok[m] * ldh + k]) : 0.f; },
-      [&](int k, int n) { return (n0 + n < ff && k < hidden) ? to_f32(wg[(size_t)(n0 + n) * hidden + k]) : 0.f; },
-      [&](int k, int n) { return (n0 + n < ff && k < hidden) ? to_f32(wu[(size_t)(n0 + n) * hidden + k]) : 0.f; },
-      s, up_s);
+  auto in = [&](int m, int k) { return (m < rows && k < hidden) ? to_f32(h[(size_t)tok[m] * ldh + k]) : 0.f; };
+  auto up = [&](int k, int n) { return (n0 + n < ff && k < hidden) ? to_f32(wu[(size_t)(n0 + n) * hidden + k]) : 0.f; };
+  if constexpr (PAIR)
+    tile_gemm_pair(
+        acc_g, acc_u, hidden, in,
+        [&](int k, int n) { return (n0 + n < ff && k < hidden) ? to_f32(wg[(size_t)(n0 + n) * hidden + k]) : 0.f; }, up, s,
+        up_s);
+  else
+    tile_gemm(acc_u, hidden, in, up, s);
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
@@ -320,7 +389,9 @@ __global__ __launch_bounds__(256) void moe_ffn1_kernel(const T* __restrict__ h, 
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx * 4 + j;
       if (n < ff)
-        act[(size_t)(row0 + m) * lda + n] = from_f32<T>(gated_value(sc * acc_g[i][j], sc * acc_u[i][j], kind, alpha, limit));
+        act[(size_t)(row0 + m) * lda + n] =
+            from_f32<T>(PAIR ? gated_value(sc * acc_g[i][j], sc * acc_u[i][j], kind, alpha, limit)
+                             : unit_value(sc * acc_u[i][j], kind));
     }
   }
 }
@@ -355,7 +426,7 @@ __global__ __launch_bounds__(256) void moe_ffn2_kernel(const T* __restrict__ act
 }
 
 // The same two products in bfloat16 on the tensor cores (mma_tile.cuh), float32 accumulation.
-template <bool VEC>
+template <bool VEC, bool PAIR>
 __global__ __launch_bounds__(128) void moe_ffn1_mma_kernel(const __nv_bfloat16* __restrict__ h, long ldh,
                                                            const __nv_bfloat16* __restrict__ w_gu,
                                                            const int* __restrict__ tiles, const int* __restrict__ meta,
@@ -364,7 +435,7 @@ __global__ __launch_bounds__(128) void moe_ffn1_mma_kernel(const __nv_bfloat16* 
                                                            __nv_bfloat16* __restrict__ act, long lda, int hidden, int ff,
                                                            int kind, float alpha, float limit) {
   __shared__ __align__(16) MmaTileSmem s;
-  __shared__ __align__(16) __nv_bfloat16 up_s[MT_STAGES][MT_N][MT_LD];
+  __shared__ __align__(16) __nv_bfloat16 up_s[PAIR ? MT_STAGES : 1][PAIR ? MT_N : 1][MT_LD];
   __shared__ int tok[MT_M];
   pdl_begin();
   if ((int)blockIdx.x >= meta[0]) return;
@@ -372,18 +443,22 @@ __global__ __launch_bounds__(128) void moe_ffn1_mma_kernel(const __nv_bfloat16* 
   const int n0 = blockIdx.y * MT_N;
   if (threadIdx.x < MT_M) tok[threadIdx.x] = threadIdx.x < rows ? row_token[row0 + threadIdx.x] : 0;
   __syncthreads();
-  const __nv_bfloat16* wg = w_gu + (size_t)e * 2 * ff * hidden;
-  const __nv_bfloat16* wu = wg + (size_t)ff * hidden;
+  const __nv_bfloat16* wg = w_gu + (size_t)e * (PAIR ? 2 : 1) * ff * hidden;
+  const __nv_bfloat16* wu = wg + (PAIR ? (size_t)ff * hidden : 0);
   float acc_g[2][4][4] = {}, acc_u[2][4][4] = {};
-  mma_tile_pair<VEC>(
-      acc_g, acc_u, hidden, [&](int m) { return m < rows ? h + (size_t)tok[m] * ldh : nullptr; },
-      [&](int n) { return n0 + n < ff ? wg + (size_t)(n0 + n) * hidden : nullptr; },
-      [&](int n) { return n0 + n < ff ? wu + (size_t)(n0 + n) * hidden : nullptr; }, s, up_s);
-  mma_for_each(acc_g, [&](int m, int n, int mi, int ni, int c) {
+  auto in = [&](int m) { return m < rows ? h + (size_t)tok[m] * ldh : nullptr; };
+  auto up = [&](int n) { return n0 + n < ff ? wu + (size_t)(n0 + n) * hidden : nullptr; };
+  if constexpr (PAIR)
+    mma_tile_pair<VEC>(
+        acc_g, acc_u, hidden, in, [&](int n) { return n0 + n < ff ? wg + (size_t)(n0 + n) * hidden : nullptr; }, up, s, up_s);
+  else
+    mma_tile<VEC>(acc_u, hidden, in, up, s);
+  mma_for_each(acc_u, [&](int m, int n, int mi, int ni, int c) {
     if (m < rows && n0 + n < ff) {
       const float sc = row_scale != nullptr ? row_scale[row0 + m] : 1.f;
       act[(size_t)(row0 + m) * lda + n0 + n] =
-          __float2bfloat16_rn(gated_value(sc * acc_g[mi][ni][c], sc * acc_u[mi][ni][c], kind, alpha, limit));
+          __float2bfloat16_rn(PAIR ? gated_value(sc * acc_g[mi][ni][c], sc * acc_u[mi][ni][c], kind, alpha, limit)
+                                   : unit_value(sc * acc_u[mi][ni][c], kind));
     }
   });
 }
@@ -414,8 +489,10 @@ __global__ __launch_bounds__(128) void moe_ffn2_mma_kernel(const __nv_bfloat16* 
 // MOE_ROWS_PASS input rows held in shared memory, and reduces over the lanes; tiles with more
 // rows take further passes (their weights then come from L2).  float32 accumulation.
 constexpr int MOE_ROWS_PASS = 4;
+// What a warp's column is: of the two input projections, of the only one, or of the output projection.
+constexpr int MOE_COL_PAIR = 0, MOE_COL_UP = 1, MOE_COL_DOWN = 2;
 
-template <bool PAIR>
+template <int COL>
 __global__ __launch_bounds__(256) void moe_rows_kernel(const __nv_bfloat16* __restrict__ x, long ldx,
                                                        const __nv_bfloat16* __restrict__ w,
                                                        const int* __restrict__ tiles, const int* __restrict__ meta,
@@ -424,6 +501,7 @@ __global__ __launch_bounds__(256) void moe_rows_kernel(const __nv_bfloat16* __re
                                                        __nv_bfloat16* __restrict__ act, long lda,
                                                        float* __restrict__ eo, int k_total, int n_total, int kind,
                                                        float alpha, float limit) {
+  constexpr bool PAIR = COL == MOE_COL_PAIR;
   extern __shared__ __align__(16) __nv_bfloat16 rows_s[];  // [MOE_ROWS_PASS][k_total]
   pdl_begin();
   if ((int)blockIdx.x >= meta[0]) return;
@@ -439,7 +517,7 @@ __global__ __launch_bounds__(256) void moe_rows_kernel(const __nv_bfloat16* __re
     __syncthreads();  // the rows of the pass before have been used
     for (int i = threadIdx.x; i < nr * k8; i += blockDim.x) {
       const int r = i / k8, c = (i - r * k8) * 8;
-      const int src = PAIR ? row_token[row0 + r0 + r] : row0 + r0 + r;
+      const int src = COL != MOE_COL_DOWN ? row_token[row0 + r0 + r] : row0 + r0 + r;
       *reinterpret_cast<uint4*>(rows_s + (size_t)r * k_total + c) = *reinterpret_cast<const uint4*>(x + (size_t)src * ldx + c);
     }
     __syncthreads();
@@ -470,9 +548,10 @@ __global__ __launch_bounds__(256) void moe_rows_kernel(const __nv_bfloat16* __re
       const float s0 = warp_sum(a0[r]);
       const float s1 = PAIR ? warp_sum(a1[r]) : 0.f;
       if (lane == 0 && n < n_total) {
-        if (PAIR) {
+        if (COL != MOE_COL_DOWN) {
           const float sc = row_scale != nullptr ? row_scale[row0 + r0 + r] : 1.f;
-          act[(size_t)(row0 + r0 + r) * lda + n] = __float2bfloat16_rn(gated_value(sc * s0, sc * s1, kind, alpha, limit));
+          act[(size_t)(row0 + r0 + r) * lda + n] =
+              __float2bfloat16_rn(PAIR ? gated_value(sc * s0, sc * s1, kind, alpha, limit) : unit_value(sc * s0, kind));
         } else
           eo[(size_t)(row0 + r0 + r) * n_total + n] = s0;
       }
@@ -480,19 +559,24 @@ __global__ __launch_bounds__(256) void moe_rows_kernel(const __nv_bfloat16* __re
   }
 }
 
-// y[t] (+)= sum_j weights[t, j] * eo[place_of[t, j]], j in order (weights null: plain sum).
+// y[t] (+)= sum_j weights[t, j] * eo[place_of[t, j]], j in order (weights null: plain sum), + sigmoid(sg[t]) *
+// shared[t] where given (shared: float32 [tokens, hidden]; sg: one logit a token, stride ldsg).
 __global__ __launch_bounds__(256) void moe_combine_kernel(const float* __restrict__ eo,
                                                           const float* __restrict__ weights,
                                                           const int* __restrict__ place_of, float* __restrict__ y,
-                                                          long ldy, int n_tokens, int hidden, int top, int add) {
+                                                          long ldy, int n_tokens, int hidden, int top, int add,
+                                                          const float* __restrict__ shared, long lds,
+                                                          const float* __restrict__ sg, long ldsg) {
   pdl_begin();
   const int t = blockIdx.x;
   if (t >= n_tokens) return;
+  const float gate = shared != nullptr ? 1.0f / (1.0f + expf(-sg[(size_t)t * ldsg])) : 0.f;
   for (int d = threadIdx.x; d < hidden; d += blockDim.x) {
     float acc = 0.f;
     for (int j = 0; j < top; ++j)
       acc = fmaf(weights != nullptr ? weights[(size_t)t * top + j] : 1.f,
                  eo[(size_t)place_of[(size_t)t * top + j] * hidden + d], acc);
+    if (shared != nullptr) acc = fmaf(gate, shared[(size_t)t * lds + d], acc);
     float* o = y + (size_t)t * ldy + d;
     *o = add ? *o + acc : acc;
   }
@@ -506,7 +590,7 @@ RL_EXPORT int rl_moe_select(const float* z, long ldz, const float* correction, i
                             int group_count, int group_keep, int score_kind, int* ids, float* weights, int* counts,
                             cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
-  if (n_experts <= 0 || n_experts > 2048 || top <= 0 || top > n_experts || score_kind < 0 || score_kind > 1) return -2;
+  if (n_experts <= 0 || n_experts > 2048 || top <= 0 || top > n_experts || score_kind < 0 || score_kind > 2) return -2;
   if (group_count < 1 || n_experts % group_count != 0 || group_keep < 1 || group_keep > group_count ||
       top > group_keep * (n_experts / group_count))
     return -3;
@@ -515,6 +599,30 @@ RL_EXPORT int rl_moe_select(const float* z, long ldz, const float* correction, i
     cudaFuncSetAttribute(rl::moe_select_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   rl::launch_pdl(rl::moe_select_kernel, (n_tokens + 3) / 4, 128, smem, stream, z, ldz, correction, n_tokens, n_experts,
                  top, group_count, group_keep, score_kind, ids, weights, counts);
+  RL_CHECK_LAUNCH();
+  return 0;
+}
+
+// Routing and layout in one launch: what rl_moe_select and rl_moe_plan leave, for at most 128 tokens (-3 beyond).  No
+// counters in global memory are used.  place_weight: null, or float32 [tokens * top] that receives the weights by place.
+RL_EXPORT int rl_moe_select_route(const float* z, long ldz, const float* correction, int n_tokens, int n_experts, int top,
+                                  int group_count, int group_keep, int score_kind, int* ids, float* weights, int* offsets,
+                                  int* tiles, int* meta, int* row_token, int* place_of, float* place_weight,
+                                  cudaStream_t stream) {
+  if (n_tokens <= 0) return 0;
+  if (n_experts <= 0 || n_experts > rl::MOE_ROUTE_MAX_EXPERTS || top <= 0 || top > n_experts || score_kind < 0 ||
+      score_kind > 2 || group_count < 1 || n_experts % group_count != 0 || group_keep < 1 || group_keep > group_count ||
+      top > group_keep * (n_experts / group_count))
+    return -2;
+  if (n_tokens > rl::MOE_ROUTE_MAX_TOKENS || (long)n_tokens * top > rl::MOE_ROUTE_MAX_PAIRS) return -3;
+  // the counts take 24 KB of static shared memory: 24 KB are left for the warps' scores (E <= 2048: one warp's fit)
+  int warps = (24 * 1024 - 64) / (3 * n_experts * (int)sizeof(float));
+  warps = warps > 32 ? 32 : warps;
+  if (warps > n_tokens) warps = n_tokens;
+  if (warps < 1) return -3;
+  rl::launch_pdl(rl::moe_select_route_kernel, 1, warps * 32, (size_t)warps * 3 * n_experts * sizeof(float), stream, z, ldz,
+                 correction, n_tokens, n_experts, top, group_count, group_keep, score_kind, ids, weights, offsets, tiles,
+                 meta, row_token, place_of, place_weight);
   RL_CHECK_LAUNCH();
   return 0;
 }
@@ -572,24 +680,27 @@ RL_EXPORT int rl_moe_max_tiles(int n_pairs, int n_experts) {
   return (n_pairs + rl::MOE_TILE_ROWS - 1) / rl::MOE_TILE_ROWS + n_experts;
 }
 
-// The experts' feed-forward on the laid-out pairs, and the weighted sum per token.
-// h: [tokens, hidden] (row stride ldh); w_gu: [experts][2][ff][hidden]; w_down:
-// [experts][hidden][ff]; act: scratch [pairs, ff] (row stride lda); eo: float32 scratch
+// The experts' feed-forward on the laid-out pairs, and (y given) the weighted sum per token.
+// h: [tokens, hidden] (row stride ldh); w_gu: [experts][2][ff][hidden] (kinds of one projection: [experts][ff][hidden]);
+// w_down: [experts][hidden][ff]; act: scratch [pairs, ff] (row stride lda); eo: float32 scratch
 // [pairs, hidden]; y: float32 [tokens, hidden] (row stride ldy), overwritten or (add) added to.
 // place_weight (by place) scales the experts' inputs, weights (by pair) their outputs; either may be null.
+// shared (or null): float32 [tokens, hidden], added times sigmoid(sg[token]).
 RL_EXPORT int rl_moe_experts(int dtype, const void* h, long ldh, const void* w_gu, const void* w_down, const int* tiles,
                              const int* meta, const int* row_token, const int* place_of, const float* weights,
-                             const float* place_weight, void* act, long lda, float* eo, float* y, long ldy, int n_tokens, int hidden, int ff,
-                             int n_experts, int top, int kind, float alpha, float limit, int add,
-                             cudaStream_t stream) {
+                             const float* place_weight, void* act, long lda, float* eo, float* y, long ldy, int n_tokens,
+                             int hidden, int ff, int n_experts, int top, int kind, float alpha, float limit, int add,
+                             const float* shared, long lds, const float* sg, long ldsg, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
-  if (hidden <= 0 || ff <= 0 || kind < 0 || kind > 3) return -2;
+  if (hidden <= 0 || ff <= 0 || kind < 0 || kind > RL_UNIT_LAST || (shared != nullptr && sg == nullptr)) return -2;
+  const bool pair = kind < RL_UNIT_FIRST;
   const int max_tiles = rl_moe_max_tiles(n_tokens * top, n_experts);
   const dim3 g1(max_tiles, (ff + rl::TG_N - 1) / rl::TG_N), g2(max_tiles, (hidden + rl::TG_N - 1) / rl::TG_N);
   if (g1.y > 65535 || g2.y > 65535) return -2;
   if (dtype == RL_F32) {
-    rl::launch_pdl(rl::moe_ffn1_kernel<float>, g1, 256, 0, stream, (const float*)h, ldh, (const float*)w_gu, tiles,
-                   meta, row_token, place_weight, (float*)act, lda, hidden, ff, kind, alpha, limit);
+    rl::launch_pdl(pair ? rl::moe_ffn1_kernel<float, true> : rl::moe_ffn1_kernel<float, false>, g1, 256, 0, stream,
+                   (const float*)h, ldh, (const float*)w_gu, tiles, meta, row_token, place_weight, (float*)act, lda, hidden,
+                   ff, kind, alpha, limit);
     rl::launch_pdl(rl::moe_ffn2_kernel<float>, g2, 256, 0, stream, (const float*)act, lda, (const float*)w_down, tiles,
                    meta, eo, hidden, ff);
   } else {
@@ -601,23 +712,25 @@ RL_EXPORT int rl_moe_experts(int dtype, const void* h, long ldh, const void* w_g
     const bool few = (long)n_tokens * top <= (long)rl::MOE_ROWS_PASS * n_experts && vec1 && vec2 && (size_t)hidden * 8 <= 48 * 1024 &&
                      (size_t)ff * 8 <= 48 * 1024;
     if (few) {
-      rl::launch_pdl(rl::moe_rows_kernel<true>, dim3(max_tiles, (ff + 7) / 8), 256,
-                     (size_t)rl::MOE_ROWS_PASS * hidden * 2, stream, (const __nv_bfloat16*)h, ldh,
-                     (const __nv_bfloat16*)w_gu, tiles, meta, row_token, place_weight, (__nv_bfloat16*)act, lda, (float*)nullptr,
-                     hidden, ff, kind, alpha, limit);
-      rl::launch_pdl(rl::moe_rows_kernel<false>, dim3(max_tiles, (hidden + 7) / 8), 256,
+      rl::launch_pdl(pair ? rl::moe_rows_kernel<rl::MOE_COL_PAIR> : rl::moe_rows_kernel<rl::MOE_COL_UP>,
+                     dim3(max_tiles, (ff + 7) / 8), 256, (size_t)rl::MOE_ROWS_PASS * hidden * 2, stream,
+                     (const __nv_bfloat16*)h, ldh, (const __nv_bfloat16*)w_gu, tiles, meta, row_token, place_weight,
+                     (__nv_bfloat16*)act, lda, (float*)nullptr, hidden, ff, kind, alpha, limit);
+      rl::launch_pdl(rl::moe_rows_kernel<rl::MOE_COL_DOWN>, dim3(max_tiles, (hidden + 7) / 8), 256,
                      (size_t)rl::MOE_ROWS_PASS * ff * 2, stream, (const __nv_bfloat16*)act, lda,
                      (const __nv_bfloat16*)w_down, tiles, meta, row_token, (const float*)nullptr, (__nv_bfloat16*)nullptr, 0L, eo, ff, hidden,
                      kind, alpha, limit);
     } else {
-    auto k1 = vec1 ? rl::moe_ffn1_mma_kernel<true> : rl::moe_ffn1_mma_kernel<false>;
+    auto k1 = pair ? (vec1 ? rl::moe_ffn1_mma_kernel<true, true> : rl::moe_ffn1_mma_kernel<false, true>)
+                   : (vec1 ? rl::moe_ffn1_mma_kernel<true, false> : rl::moe_ffn1_mma_kernel<false, false>);
     auto k2 = vec2 ? rl::moe_ffn2_mma_kernel<true> : rl::moe_ffn2_mma_kernel<false>;
     // three stages of three operands are 46 KB a block: with the common half-and-half split of an
     // SM's memory two blocks fit, with all of it as shared memory four (the registers' limit)
-    static bool carved[4] = {false, false, false, false};
-    if (!carved[vec1]) {
+    static bool carved[6] = {false, false, false, false, false, false};
+    const int c1 = (pair ? 0 : 4) + (vec1 ? 1 : 0);
+    if (!carved[c1]) {
       cudaFuncSetAttribute(k1, cudaFuncAttributePreferredSharedMemoryCarveout, (int)cudaSharedmemCarveoutMaxShared);
-      carved[vec1] = true;
+      carved[c1] = true;
     }
     if (!carved[2 + vec2]) {
       cudaFuncSetAttribute(k2, cudaFuncAttributePreferredSharedMemoryCarveout, (int)cudaSharedmemCarveoutMaxShared);
@@ -629,8 +742,9 @@ RL_EXPORT int rl_moe_experts(int dtype, const void* h, long ldh, const void* w_g
                          tiles, meta, eo, hidden, ff);
     }
   }
-  rl::launch_pdl(rl::moe_combine_kernel, n_tokens, 256, 0, stream, (const float*)eo, weights, place_of, y, ldy,
-                 n_tokens, hidden, top, add);
+  if (y != nullptr)
+    rl::launch_pdl(rl::moe_combine_kernel, n_tokens, 256, 0, stream, (const float*)eo, weights, place_of, y, ldy, n_tokens,
+                   hidden, top, add, shared, lds, sg, ldsg);
   RL_CHECK_LAUNCH();
   return 0;
 }

@@ -11,6 +11,7 @@
 #define RL_ACT_NONE 0
 #define RL_ACT_GELU_TANH 1
 #define RL_ACT_GELU_ERF 2
+#define RL_ACT_RELU_SQUARED 3
 
 namespace rl {
 namespace tc {
@@ -29,6 +30,10 @@ __device__ __forceinline__ float act_fn(float u, int act) {
     return 0.5f * u * (1.0f + t);
   }
   if (act == RL_ACT_GELU_ERF) return 0.5f * u * (1.0f + erff(u * 0.7071067811865476f));
+  if (act == RL_ACT_RELU_SQUARED) {
+    const float r = fmaxf(u, 0.f);
+    return r * r;
+  }
   return u;
 }
 

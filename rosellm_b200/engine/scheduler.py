@@ -170,10 +170,10 @@ class Scheduler:
     def _pages_to_hold(self, n_tokens: int) -> list[int]:
         out = []
         for g in self.cache.groups:
-            if g.spec.window is None:
+            if not g.spec.bounded:
                 out.append(pages_for(n_tokens, self.cache.page_size))
             else:
-                span = min(n_tokens, g.spec.window + self.prefill_chunk_size)
+                span = min(n_tokens, g.spec.reach + self.prefill_chunk_size)
                 out.append(pages_for(span, self.cache.page_size) + 1)
         return out
 

@@ -3,6 +3,7 @@ from . import lebedra  # registers Lebedra
 from . import porovik  # registers Porovik
 from . import fikevik  # registers Fikevik
 from . import soporax  # registers Soporax
+from . import vebotar  # registers Vebotar
 from .model import Layer, Model, named_params_of_spec
 
-__all__ = ["Layer", "Model", "named_params_of_spec", "gpt2", "lebedra", "porovik", "fikevik", "soporax"]
+__all__ = ["Layer", "Model", "named_params_of_spec", "gpt2", "lebedra", "porovik", "fikevik", "soporax", "vebotar"]

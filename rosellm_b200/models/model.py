@@ -111,6 +111,9 @@ class Model:
         # what is added to the stream between runs of layers: the parts, and per position of the run order the
         # (part, arguments) that come right before it
         self.stream_parts = [build_part("stream_input", ps) for ps in spec.stream_parts]
+        if any(si.before > 0 for si in spec.stream_inputs) and any(getattr(l.block, "keeps_copies", False) for l in self.layers):
+            raise ValueError("stream inputs between runs add to one row a token: they cannot go between layers that "
+                             "keep the stream in several copies")
         self._stream_before: dict[int, list] = {}
         for si in spec.stream_inputs:
             self._stream_before.setdefault(si.before, []).append((self.stream_parts[si.part], dict(si.args)))
@@ -137,11 +140,15 @@ class Model:
                 continue
             for name, part in self.layers[e.layer].parts.items():
                 own = part.cache_spec()
-                if own is not None and own != out.get(_cache_key(e.cache_layer, name)):
+                if own is None:
+                    continue
+                key = _cache_key(e.cache_layer, name)
+                if key not in out or not own.same_rows(out[key]):
                     raise ValueError(
                         f"run_order[{pos}]: {name!r} of layer {e.layer} reads the cache of layer {e.cache_layer}, "
                         "whose geometry differs from what it expects"
                     )
+                out[key] = out[key].covering(own)  # pages stay as long as any reader sees into them
         return out
 
     def state_specs(self) -> dict:

@@ -15,8 +15,8 @@ import torch
 from . import build
 
 F32, BF16 = 0, 1
-ACT_NONE, ACT_GELU_TANH, ACT_GELU_ERF = 0, 1, 2
-ACTIVATIONS = {"none": ACT_NONE, "gelu_tanh": ACT_GELU_TANH, "gelu_erf": ACT_GELU_ERF}
+ACT_NONE, ACT_GELU_TANH, ACT_GELU_ERF, ACT_RELU_SQUARED = 0, 1, 2, 3
+ACTIVATIONS = {"none": ACT_NONE, "gelu_tanh": ACT_GELU_TANH, "gelu_erf": ACT_GELU_ERF, "relu_squared": ACT_RELU_SQUARED}
 
 STATUS_BITS = {
     1: "a token id outside the embedding table",
@@ -166,7 +166,9 @@ def _lib() -> ctypes.CDLL:
         lib.rl_moe_select.argtypes = [P, L, P, I, I, I, I, I, I, P, P, P, P]
         lib.rl_moe_plan.argtypes = [P, P, P, P, P, P, P, P, P, P, I, I, I, P]
         lib.rl_moe_max_tiles.argtypes = [I, I]
-        lib.rl_moe_experts.argtypes = [I, P, L, P, P, P, P, P, P, P, P, P, L, P, P, L, I, I, I, I, I, I, F, F, I, P]
+        lib.rl_moe_experts.argtypes = [I, P, L, P, P, P, P, P, P, P, P, P, L, P, P, L, I, I, I, I, I, I, F, F, I, P, L, P, L, P]
+        lib.rl_moe_select_route.argtypes = [P, L, P, I, I, I, I, I, I, P, P, P, P, P, P, P, P, P]
+        lib.rl_hyper_step.argtypes = [I, P, L, L, P, L, P, L, P, P, P, P, F, P, L, P, L, I, I, I, P, P, P, I, P, L, P, L, P]
         lib.rl_embed_pair.argtypes = [I, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, P, P, P, I, P]
         lib.rl_rmsnorm_add_norm.argtypes = [I, P, L, P, P, L, P, P, L, I, I, F, F, P]
         lib.rl_recurrence.argtypes = [I, I, P, L, I, I, I, I, I, I, P, P, P, I, P, P, P, L, P, P, P, P, I, I, I, I, I, F, F, F,
@@ -174,8 +176,8 @@ def _lib() -> ctypes.CDLL:
         lib.rl_recurrence_record.argtypes = [I, I, I, P, P, P]
         lib.rl_bias_attention_shape.argtypes = [I, I, P, P]
         lib.rl_bias_attention.argtypes = [I, I, P, L, P, L, P, P, L, P, P, P, P, I, I, P, I, P, L, I, I, I, I, I, I, I, I,
-                                          F, F, I, P, P, I, P, P, I, I, P, P, I, P]
-        lib.rl_qkv_norm_rotate.argtypes = [P, L, P, L, P, L, P, P, P, P, I, I, I, I, I, I, I, I, F,
+                                          F, F, I, P, P, I, P, P, I, I, P, P, I, I, I, P, F, F, P]
+        lib.rl_qkv_norm_rotate.argtypes = [P, L, P, L, P, L, P, P, P, P, I, I, I, I, I, I, I, F, I, I, F,
                                            I, P, P, L, P, P, I, I, I, I, P, P]
         lib.rl_stream_inject.argtypes = [P, L, P, P, L, P, L, I, I, P]
         lib.rl_gate_mul.argtypes = [I, P, L, P, L, I, I, P]
@@ -189,7 +191,8 @@ def _lib() -> ctypes.CDLL:
                      "rl_token_gate", "rl_moe_select", "rl_moe_plan", "rl_moe_max_tiles", "rl_moe_experts", "rl_embed_pair",
                      "rl_rmsnorm_add_norm", "rl_recurrence", "rl_recurrence_record", "rl_bias_attention_shape", "rl_bias_attention",
                      "rl_bias_kv_store", "rl_qkv_norm_rotate", "rl_gated_join_norm", "rl_stream_inject", "rl_gate_mul",
-                     "rl_moe_table_select", "rl_stream_inject_norm", "rl_moe_table_route"):
+                     "rl_moe_table_select", "rl_stream_inject_norm", "rl_moe_table_route",
+                     "rl_moe_select_route", "rl_hyper_step"):
             getattr(lib, name).restype = I
         for name in ("rl_copy_to_device", "rl_event_record", "rl_embed", "rl_layernorm", "rl_gemm_simt", "rl_gemm_tc", "rl_gemm_tc_sample", "rl_gemm_tc_cut", "rl_gemm_tc_rows", "rl_gemm_tc_rows_fits",
                      "rl_gemm_rows_smem", "rl_gemm_rows_smem_fits",
@@ -1102,6 +1105,7 @@ def head_linear(inp, w, out, *, n_tokens: int, n_heads: int, k: int, n: int, in_
 # ---- gated feed-forward, token-gated input, mixture of experts ---------------------------------
 
 GATES = {"relu": 0, "silu": 1, "gelu_tanh": 2, "clamped_swish": 3}
+UNITS = {"relu_squared": 4}  # activations of layers with one input projection (csrc/gated_act.cuh)
 
 
 def gated_act(gu, out, *, width: int, up_at: int, gate: int, alpha: float = 1.0, limit: float = 0.0) -> None:
@@ -1174,14 +1178,15 @@ def moe_max_tiles(n_pairs: int, n_experts: int) -> int:
     return int(_lib().rl_moe_max_tiles(n_pairs, n_experts))
 
 
-MOE_SCORES = {"softmax": 0, "sigmoid": 1}
+MOE_SCORES = {"softmax": 0, "sigmoid": 1, "chosen_softmax": 2}
 
 
 def moe_select(z, correction, *, top: int, group_count: int, group_keep: int, ids, weights, counts,
                score: int = 0) -> None:
     """Routing of every row of the float32 router logits ``z`` [tokens, experts]: see csrc/moe.cu.
     ``ids`` int32 and ``weights`` float32 [tokens * top]; ``counts`` int32 [experts], zero on entry.
-    ``score``: 0 softmax over the experts, 1 each expert's sigmoid."""
+    ``score``: 0 softmax over the experts, 1 each expert's sigmoid, 2 the choice by the logits and the softmax over the
+    chosen experts' logits alone."""
     _need(z, "z", torch.float32, contiguous=False)
     n, n_experts = z.shape
     for t, name, dt in ((ids, "ids", torch.int32), (weights, "weights", torch.float32), (counts, "counts", torch.int32)):
@@ -1193,6 +1198,35 @@ def moe_select(z, correction, *, top: int, group_count: int, group_keep: int, id
     if rc in (-2, -3):
         raise KernelError(f"moe_select: {n_experts} experts, top {top}, {group_keep} of {group_count} groups not taken")
     _ok(rc, "moe_select")
+
+
+MOE_ROUTE_MAX_TOKENS = 128  # csrc/moe.cu: MOE_ROUTE_MAX_TOKENS
+
+
+def moe_select_route(z, correction, *, top: int, group_count: int, group_keep: int, score: int, ids, weights, offsets,
+                     tiles, meta, row_token, place_of, place_weight=None) -> None:
+    """``moe_select`` and ``moe_plan`` in one launch, for at most ``MOE_ROUTE_MAX_TOKENS`` tokens: the same ``ids``,
+    ``weights``, ``offsets``, ``tiles``, ``meta``, ``row_token``, ``place_of`` and (given) ``place_weight``."""
+    _need(z, "z", torch.float32, contiguous=False)
+    n, n_experts = z.shape
+    _need(weights, "weights", torch.float32)
+    for t, name in ((ids, "ids"), (offsets, "offsets"), (tiles, "tiles"), (meta, "meta"), (row_token, "row_token"),
+                    (place_of, "place_of")):
+        _need(t, name, torch.int32)
+    for t, name in ((correction, "correction"), (place_weight, "place_weight")):
+        if t is not None:
+            _need(t, name, torch.float32)
+    if min(ids.numel(), weights.numel(), row_token.numel(), place_of.numel()) < n * top or offsets.numel() < n_experts + 1 \
+            or tiles.numel() < 3 * moe_max_tiles(n * top, n_experts) \
+            or (place_weight is not None and place_weight.numel() < n * top):
+        raise KernelError("moe_select_route: the outputs are too small")
+    rc = _lib().rl_moe_select_route(_ptr(z), z.stride(0), _ptr(correction), n, n_experts, top, group_count, group_keep,
+                                    int(score), _ptr(ids), _ptr(weights), _ptr(offsets), _ptr(tiles), _ptr(meta),
+                                    _ptr(row_token), _ptr(place_of), _ptr(place_weight), _stream())
+    if rc in (-2, -3):
+        raise KernelError(f"moe_select_route: {n} tokens, {n_experts} experts, top {top}, {group_keep} of {group_count} "
+                          "groups not taken")
+    _ok(rc, "moe_select_route")
 
 
 def moe_table_select(token_ids, table, *, n_experts: int, weight: float, ids, weights, counts, feedback=None) -> None:
@@ -1256,9 +1290,13 @@ def moe_plan(ids, counts, fill, offsets, tiles, meta, row_token, place_of, *, n_
 
 
 def moe_experts(h, w_gate_up, w_down, tiles, meta, row_token, place_of, weights, act, eo, y, *, n_experts: int, top: int,
-                ff: int, gate: int, alpha: float, limit: float, add: bool, place_weight=None) -> None:
-    """The experts' gated feed-forward on the laid-out pairs and the weighted sum per token into
-    ``y`` float32 [tokens, hidden] (``add``: added to it).  ``weights`` (by pair) weight the experts'
+                ff: int, gate: int, alpha: float, limit: float, add: bool, place_weight=None, shared=None,
+                shared_gate=None) -> None:
+    """The experts' feed-forward on the laid-out pairs and the weighted sum per token into
+    ``y`` float32 [tokens, hidden] (``add``: added to it; ``None``: no sum, the experts' outputs stay in ``eo`` by place).
+    ``gate``: a code of ``GATES`` (two input projections) or of ``UNITS`` (one: ``w_gate_up`` is then [experts * ff,
+    hidden]).  ``shared`` float32 [tokens, hidden] and ``shared_gate`` float32 [tokens] (a column of a matrix will do):
+    added times the logit's sigmoid.  ``weights`` (by pair) weight the experts'
     outputs; ``place_weight`` (by place, from ``moe_plan``) their inputs instead; either may be ``None``.  ``w_gate_up`` [experts * 2 * ff, hidden]
     (per expert: gate rows, then up rows), ``w_down`` [experts * hidden, ff]."""
     _need(h, "h", contiguous=False)
@@ -1266,18 +1304,101 @@ def moe_experts(h, w_gate_up, w_down, tiles, meta, row_token, place_of, weights,
     _need(w_down, "w_down", h.dtype)
     _need(act, "act", h.dtype, contiguous=False)
     _need(eo, "eo", torch.float32)
-    _need(y, "y", torch.float32, contiguous=False)
     n, hidden = h.shape
-    if tuple(w_gate_up.shape) != (n_experts * 2 * ff, hidden) or tuple(w_down.shape) != (n_experts * hidden, ff) \
-            or act.shape[0] < n * top or act.shape[1] < ff or eo.numel() < n * top * hidden or tuple(y.shape) != (n, hidden):
+    if y is not None:
+        _need(y, "y", torch.float32, contiguous=False)
+    if tuple(w_gate_up.shape) != (n_experts * (2 if gate in GATES.values() else 1) * ff, hidden) \
+            or tuple(w_down.shape) != (n_experts * hidden, ff) or act.shape[0] < n * top or act.shape[1] < ff \
+            or eo.numel() < n * top * hidden or (y is not None and tuple(y.shape) != (n, hidden)):
         raise KernelError("moe_experts: shapes do not fit")
+    if shared is not None:
+        _need(shared, "shared", torch.float32, contiguous=False)
+        _need(shared_gate, "shared_gate", torch.float32, contiguous=False)
+        if tuple(shared.shape) != (n, hidden) or shared.stride(1) != 1 or shared_gate.shape != (n,):
+            raise KernelError("moe_experts: the shared feed-forward's output or gate has another shape")
     rc = _lib().rl_moe_experts(_code(h), _ptr(h), h.stride(0), _ptr(w_gate_up), _ptr(w_down), _ptr(tiles), _ptr(meta),
                                _ptr(row_token), _ptr(place_of), _ptr(weights), _ptr(place_weight), _ptr(act), act.stride(0), _ptr(eo), _ptr(y),
-                               y.stride(0), n, hidden, ff, n_experts, top, gate, float(alpha), float(limit), int(add),
-                               _stream())
+                               0 if y is None else y.stride(0), n, hidden, ff, n_experts, top, gate, float(alpha), float(limit),
+                               int(add), _ptr(shared), 0 if shared is None else shared.stride(0), _ptr(shared_gate),
+                               0 if shared is None else shared_gate.stride(0), _stream())
     _ok(rc, "moe_experts")
     global _launches
-    _launches += 2
+    _launches += 2 if y is not None else 1
+
+
+class ExpertSum:
+    """A mixture of experts' result not yet summed: the experts' outputs by place (``eo`` float32 [tokens * top, hidden]),
+    the pairs' weights (or ``None``), where each pair's output lies, and the output and gate logits of a feed-forward
+    that every token passes beside its experts (or ``None``).  ``hyper_step`` takes it in place of a sublayer's output."""
+
+    def __init__(self, eo, weights, place_of, top: int, shared=None, shared_gate=None) -> None:
+        self.eo, self.weights, self.place_of, self.top = eo, weights, place_of, int(top)
+        self.shared, self.shared_gate = shared, shared_gate
+
+
+HYPER_MAX_COPIES, HYPER_MAX_WIDTH = 16, 12000  # csrc/hyper_streams.cu
+
+
+def hyper_step(x, y, *, copies: int, write=None, x_new=None, read=None, gamma=None, eps: float = 0.0, h=None, total=None) -> None:
+    """What lies between two sublayers of a stream kept in ``copies`` copies (csrc/hyper_streams.cu), in one launch.
+
+    ``x`` float32: the copies [tokens, copies, width], or [tokens, width]: one row that all copies equal.  ``write``
+    (mix [copies, copies] indexed [from, to], out [copies]): every new copy is its mix of the old ones plus out times
+    ``y`` (float32 [tokens, width], or an ``ExpertSum``), stored in ``x_new`` [tokens, copies, width] (may be ``x``;
+    ``None``: not stored).  Then either ``read`` [copies], ``gamma`` [width], ``eps``: ``h`` [tokens, width] receives the
+    RMS norm of the weighted sum of the copies times ``gamma``; or ``total`` float32 [tokens, width] their plain sum."""
+    _need(x, "x", torch.float32)
+    n, width = x.shape[0], x.shape[-1]
+    one_row = x.dim() == 2
+    if not one_row and x.shape[1] != copies:
+        raise KernelError("hyper_step: x holds another number of copies")
+    mix = out_w = None
+    if write is not None:
+        mix, out_w = write
+        _need(mix, "mix", torch.float32)
+        _need(out_w, "out", torch.float32)
+        if mix.numel() != copies * copies or out_w.numel() != copies:
+            raise KernelError("hyper_step: the write's weights have another size")
+    elif x_new is not None or y is not None:
+        raise KernelError("hyper_step: nothing is written without the write's weights")
+    if x_new is not None:
+        _need(x_new, "x_new", torch.float32)
+        if tuple(x_new.shape) != (n, copies, width):
+            raise KernelError("hyper_step: x_new has another shape")
+    yp, ldy = None, 0
+    ex = (None, None, None, 0, None, 0, None, 0)
+    if isinstance(y, ExpertSum):
+        _need(y.eo, "y.eo", torch.float32)
+        _need(y.place_of, "y.place_of", torch.int32)
+        if y.eo.numel() < n * y.top * width or y.place_of.numel() < n * y.top:
+            raise KernelError("hyper_step: the experts' outputs are too small")
+        if y.shared is not None and (tuple(y.shared.shape) != (n, width) or y.shared.stride(1) != 1 or y.shared_gate.shape != (n,)):
+            raise KernelError("hyper_step: the shared feed-forward's output or gate has another shape")
+        ex = (_ptr(y.eo), _ptr(y.weights), _ptr(y.place_of), y.top, _ptr(y.shared), 0 if y.shared is None else y.shared.stride(0),
+              _ptr(y.shared_gate), 0 if y.shared is None else y.shared_gate.stride(0))
+    elif write is not None:
+        _need(y, "y", torch.float32, contiguous=False)
+        if tuple(y.shape) != (n, width) or y.stride(1) != 1:
+            raise KernelError("hyper_step: y has another shape")
+        yp, ldy = _ptr(y), y.stride(0)
+    if (read is None) == (total is None):
+        raise KernelError("hyper_step: the copies are read by the next sublayer, or summed")
+    if read is not None:
+        _need(read, "read", torch.float32)
+        _need(gamma, "gamma", torch.float32)
+        _need(h, "h")
+        if read.numel() != copies or gamma.numel() != width or tuple(h.shape) != (n, width):
+            raise KernelError("hyper_step: the read's weights or its output have another size")
+    else:
+        _need(total, "total", torch.float32)
+        if tuple(total.shape) != (n, width):
+            raise KernelError("hyper_step: the sum has another shape")
+    rc = _lib().rl_hyper_step(F32 if h is None else _code(h), _ptr(x), x.stride(0), 0 if one_row else width, _ptr(x_new),
+                              copies * width, yp, ldy, _ptr(mix), _ptr(out_w), _ptr(read), _ptr(gamma), float(eps), _ptr(h),
+                              width, _ptr(total), width, n, copies, width, *ex, _stream())
+    if rc in (-2, -3):
+        raise KernelError(f"hyper_step: {copies} copies of {width} entries not taken (at most {HYPER_MAX_COPIES}, {HYPER_MAX_WIDTH})")
+    _ok(rc, "hyper_step")
 
 
 # ---- embedding with a table chosen by pairs of tokens ------------------------------------------
@@ -1403,9 +1524,11 @@ def recurrence(mode: int, proj, offsets: dict, state, out, q_start, slots, prep,
 BIAS_ATTENTION_TENSOR_CORES = True  # prompt portions in bfloat16 on mma.sync (off: the CUDA-core kernel throughout)
 
 
-def bias_attention_tensor_cores(dtype: torch.dtype, dk: int, dv: int) -> bool:
-    """Whether ``bias_attention`` may be asked for its tensor-core form for prompt portions."""
-    return BIAS_ATTENTION_TENSOR_CORES and dtype == torch.bfloat16 and dk <= 128 and dv <= 128
+def bias_attention_tensor_cores(dtype: torch.dtype, dk: int, dv: int, maps: int = 1) -> bool:
+    """Whether ``bias_attention`` may be asked for its tensor-core form for prompt portions (two maps: where the cache
+    rows can be copied in 16-byte pieces)."""
+    return (BIAS_ATTENTION_TENSOR_CORES and dtype == torch.bfloat16 and dk <= 128 and dv <= 128
+            and (maps == 1 or (dk % 8 == 0 and dv % 8 == 0)))
 
 
 def bias_attention_async(on: bool) -> None:
@@ -1418,11 +1541,12 @@ def bias_attention_async(on: bool) -> None:
     lib.rl_bias_attention_async(int(bool(on)))
 
 
-def bias_attention_shape(heads_per_group: int, tensor_cores: bool = False) -> tuple[int, int]:
+def bias_attention_shape(heads_per_group: int, tensor_cores: bool = False, maps: int = 1) -> tuple[int, int]:
     """(heads a block, tokens a block) of ``bias_attention``'s prompt tiles for so many query heads a
-    key/value head: of the 32 rows of the CUDA-core kernel's blocks, or the 64 of the tensor-core kernel's."""
+    key/value head: of the 32 rows of the CUDA-core kernel's blocks (with two maps they are 16 pairs of rows), or the 64
+    (pairs of) rows of the tensor-core kernel's."""
     hb, tt = c_int(0), c_int(0)
-    if _lib().rl_bias_attention_shape(int(heads_per_group), 64 if tensor_cores else 32, ctypes.byref(hb), ctypes.byref(tt)) != 0:
+    if _lib().rl_bias_attention_shape(int(heads_per_group), 64 if tensor_cores else 32 // maps, ctypes.byref(hb), ctypes.byref(tt)) != 0:
         raise KernelError("bias_attention_shape: heads per group must be positive")
     return hb.value, tt.value
 
@@ -1461,7 +1585,8 @@ def bias_attention(q, gate, pool, block_table, q_start, kv_len, slots, out, *, n
                    scale: float, slopes=None, temp_coef: float = 0.0, temp_every: int = 0, tiles=None, n_tiles: int = 0,
                    tile_tokens: int = 16, decode_reqs=None, n_decode: int = 0, max_pos: int, n_splits: int = 1, part_o=None,
                    part_ml=None, tensor_cores: bool = False, window: int = 0, head_scale=None, sink=None,
-                   gate_per_head: bool = False) -> None:
+                   gate_per_head: bool = False, chunk: int = 0, maps: int = 1, diff_lambda=None, diff_eps: float = 0.0,
+                   diff_mul: float = 1.0) -> None:
     """Causal attention of the step's queries over the cached rows (csrc/bias_attention.cu).
     ``tensor_cores``: prompt portions on mma.sync (bfloat16 pool and output, sizes up to 128; the tiles cut as
     ``bias_attention_shape(.., True)`` says).
@@ -1471,13 +1596,21 @@ def bias_attention(q, gate, pool, block_table, q_start, kv_len, slots, out, *, n
     with a row stride; ``out`` [tokens, heads * dv] float32 or bfloat16; ``slopes`` float32 [heads] or ``None``.
     ``window`` > 0: a query sees itself and the ``window - 1`` keys before it; ``head_scale`` float32 [heads]: a
     further factor of every score of a head; ``sink`` float32 [heads]: one more term exp(sink[h]) in the softmax's
-    denominator (no key, no value, not scaled); ``gate_per_head``: ``gate`` is [tokens, heads], one logit a head."""
+    denominator (no key, no value, not scaled); ``gate_per_head``: ``gate`` is [tokens, heads], one logit a head.
+    ``chunk`` > 0: a query sees only the keys of its own chunk of so many positions, counted from the sequence's start.
+    ``maps`` 2: differential attention: ``q`` [tokens, heads * 2 * dk] and two keys a cached row, two softmax maps a head
+    over the same values, ``out`` = rmsnorm(a_1 - diff_lambda a_2; ``diff_eps``) * ``diff_mul`` per head (``diff_lambda``
+    a float32 device scalar); the parts' scratch has an entry a map."""
     _need(q, "q", torch.float32, contiguous=False)
     _need(out, "out", contiguous=False)
     _need(pool, "pool")
     _, planes, n_kv, page_size, row = pool.shape
-    if planes != 1 or q.shape[1] != n_heads * dk or out.shape[1] != n_heads * dv or q.stride(1) != 1 or out.stride(1) != 1:
+    if planes != 1 or q.shape[1] != n_heads * maps * dk or out.shape[1] != n_heads * dv or q.stride(1) != 1 or out.stride(1) != 1:
         raise KernelError("bias_attention: shapes do not fit")
+    if maps != 1:
+        if maps != 2 or gate is not None or sink is not None or out.dtype != pool.dtype or v_at < 2 * dk:
+            raise KernelError("bias_attention: two maps take no gate and no sink, a cache of the output's type, and two keys a row")
+        _need(diff_lambda, "diff_lambda", torch.float32)
     if gate is not None:
         _need(gate, "gate", torch.float32, contiguous=False)
         if gate.shape[1] != (n_heads if gate_per_head else n_heads * dv) or gate.stride(1) != 1:
@@ -1492,7 +1625,8 @@ def bias_attention(q, gate, pool, block_table, q_start, kv_len, slots, out, *, n
         n_splits = 1
     if n_splits > 1:
         if part_o is None or part_ml is None or part_o.dtype != torch.float32 or part_ml.dtype != torch.float32 \
-                or part_o.numel() < n_decode * n_heads * n_splits * dv or part_ml.numel() < n_decode * n_heads * n_splits * 2:
+                or part_o.numel() < n_decode * n_heads * maps * n_splits * dv \
+                or part_ml.numel() < n_decode * n_heads * maps * n_splits * 2:
             raise KernelError("bias_attention: the parts' scratch is missing or too small")
         _launches += 1
     rc = _lib().rl_bias_attention(_code(pool), _code(out), _ptr(q), q.stride(0), _ptr(gate), 0 if gate is None else gate.stride(0),
@@ -1501,10 +1635,11 @@ def bias_attention(q, gate, pool, block_table, q_start, kv_len, slots, out, *, n
                                   _ptr(out), out.stride(0), n_heads, n_kv, dk, dv, int(v_at), row, page_size,
                                   min(block_table.shape[1], -(-max_pos // page_size)), float(scale), float(temp_coef),
                                   int(temp_every), _ptr(slopes), _ptr(status_word(out.device)), int(n_splits), _ptr(part_o),
-                                  _ptr(part_ml), int(bool(tensor_cores) and bias_attention_tensor_cores(pool.dtype, dk, dv)
+                                  _ptr(part_ml), int(bool(tensor_cores) and bias_attention_tensor_cores(pool.dtype, dk, dv, maps)
                                                      and out.dtype == torch.bfloat16), int(window), _ptr(head_scale),
-                                  _ptr(sink), int(bool(gate_per_head)), _stream())
-    if rc in (-2, -3, -4):
+                                  _ptr(sink), int(bool(gate_per_head)), int(chunk), int(maps), _ptr(diff_lambda),
+                                  float(diff_eps), float(diff_mul), _stream())
+    if rc in (-2, -3, -4, -5):
         raise KernelError(f"bias_attention: sizes not taken (code {rc}: key and value sizes up to 256; tiles a multiple "
                           "of the tokens a block takes)")
     _ok(rc, "bias_attention")
@@ -1521,15 +1656,21 @@ class QkvCache:
 
 def qkv_norm_rotate(q, k, v, positions, *, n_heads: int, n_kv: int, dk: int, dv: int, eps: float, q_norm=None, k_norm=None,
                     freq=None, rot_dims: int = 0, unit_values: bool = False, unit_qk: bool = False,
-                    cache: "QkvCache | None" = None) -> None:
+                    cache: "QkvCache | None" = None, maps: int = 1, rot_mult: float = 1.0) -> None:
     """In place on float32 views (row strides allowed): every head of ``q`` [tokens, heads * dk] and ``k``
     [tokens, kv heads * dk] divided by its root mean square and multiplied by ``q_norm`` / ``k_norm`` (float32
     [dk], both or neither), then its first ``rot_dims`` entries turned in neighbouring pairs by position *
     ``freq[i]``; with ``unit_values`` every head of ``v`` [tokens, kv heads * dv] divided by its root mean square;
     with ``unit_qk`` (and no weights) every head of q and k divided by its root mean square and left so.
     ``cache`` (a ``QkvCache``): keys and values go into their cache pages as ``bias_kv_store`` would put them (and
-    are not written back in place): no store kernel is needed behind this one."""
-    for t, name, width in ((q, "q", n_heads * dk), (k, "k", n_kv * dk), (v, "v", n_kv * dv)):
+    are not written back in place): no store kernel is needed behind this one.  ``maps``: vectors of ``dk`` entries a
+    head of q and a key/value head of k, each treated by itself.  ``rot_mult``: a factor of the cosines and sines.
+    ``k`` and ``v`` ``None``: queries alone (a layer that reads another layer's cache)."""
+    if (k is None) != (v is None) or (k is None and (cache is not None or unit_values)):
+        raise KernelError("qkv_norm_rotate: keys and values are given together, and a cache target needs them")
+    for t, name, width in ((q, "q", n_heads * maps * dk), (k, "k", n_kv * maps * dk), (v, "v", n_kv * dv)):
+        if t is None:
+            continue
         _need(t, name, torch.float32, contiguous=False)
         if t.shape[1] != width or t.stride(1) != 1 or t.shape[0] != q.shape[0]:
             raise KernelError(f"qkv_norm_rotate: {name} has another shape")
@@ -1548,14 +1689,16 @@ def qkv_norm_rotate(q, k, v, positions, *, n_heads: int, n_kv: int, dk: int, dv:
         _need(pool, "cache.pool")
         _need(cache.block_table, "cache.block_table", torch.int32)
         _, planes, heads, page_size, row = pool.shape
-        if planes != 1 or heads != n_kv or cache.v_at < dk or cache.v_at + dv > row:
+        if planes != 1 or heads != n_kv or cache.v_at < maps * dk or cache.v_at + dv > row:
             raise KernelError("qkv_norm_rotate: the cache's rows do not fit the keys and values")
         cx = (_code(pool), _ptr(pool), _ptr(cache.block_table), cache.block_table.stride(0), _ptr(cache.req_of_token),
               _ptr(cache.slots), int(cache.v_at), row, page_size,
               min(cache.block_table.shape[1], -(-cache.max_pos // page_size)), _ptr(status_word(pool.device)))
-    rc = _lib().rl_qkv_norm_rotate(_ptr(q), q.stride(0), _ptr(k), k.stride(0), _ptr(v), v.stride(0), _ptr(q_norm), _ptr(k_norm),
-                                   _ptr(freq) if rot_dims else None, _ptr(positions), q.shape[0], n_heads, n_kv, dk, dv,
-                                   int(rot_dims), int(bool(unit_values)), int(bool(unit_qk)), float(eps), *cx, _stream())
+    rc = _lib().rl_qkv_norm_rotate(_ptr(q), q.stride(0), _ptr(k), 0 if k is None else k.stride(0), _ptr(v),
+                                   0 if v is None else v.stride(0), _ptr(q_norm), _ptr(k_norm),
+                                   _ptr(freq) if rot_dims else None, _ptr(positions), q.shape[0], n_heads, n_kv, int(maps), dk, dv,
+                                   int(rot_dims), float(rot_mult), int(bool(unit_values)), int(bool(unit_qk)), float(eps), *cx,
+                                   _stream())
     if rc == -2:
         raise KernelError("qkv_norm_rotate: sizes not taken (an even number of turned entries, at most the key size; "
                           "both norms or neither)")

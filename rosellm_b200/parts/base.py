@@ -31,15 +31,17 @@ Categories and the signature of ``forward``:
                    in ``ctx.extras["normed_ahead"]`` if the layer's block says it takes it);
                    ``keep_embedding(ctx, x)`` is called right after the embedding for a part none of whose
                    inputs comes first.
+``connection``     how a sublayer reads and writes a stream of another form than one row a token (weights that a
+                   block arranging such a stream uses: ``parts/hyper.py``).
 """
 from __future__ import annotations
 
-from dataclasses import dataclass
+from dataclasses import dataclass, replace
 from typing import Any, Callable
 
 import torch
 
-CATEGORIES = ("embedding", "position", "norm", "mixer", "feed_forward", "block", "head", "stream_input")
+CATEGORIES = ("embedding", "position", "norm", "mixer", "feed_forward", "block", "head", "stream_input", "connection")
 
 _PARTS: dict[tuple[str, str], type] = {}
 
@@ -99,6 +101,9 @@ class ParamSpec:
 class KVCacheSpec:
     """Keys and values in pages.  ``window``: how many latest keys a query sees
     (``None``: all of them); older pages are given back while the request lives.
+    ``chunks``: sizes of chunks, counted from the sequence's first token, of which a query sees its own alone.
+    A spec with a window and chunks, or with chunks of several sizes, is that of a cache read by several layers: a
+    page is kept while any of them sees into it (``covering``).
     ``planes``: 2 for keys and values kept apart; 1 where one cached row per token serves as
     both (a latent that the mixer's queries and outputs are projected onto)."""
 
@@ -106,6 +111,37 @@ class KVCacheSpec:
     head_dim: int
     window: int | None = None
     planes: int = 2
+    chunks: tuple[int, ...] = ()
+
+    @property
+    def bounded(self) -> bool:
+        """Whether keys are ever out of every later query's sight while the request lives."""
+        return self.window is not None or bool(self.chunks)
+
+    @property
+    def reach(self) -> int:
+        """The most keys a query sees (of a bounded spec)."""
+        return max((self.window or 0, *self.chunks))
+
+    def first_key(self, pos: int) -> int:
+        """The earliest key that a query at ``pos`` or later sees."""
+        if not self.bounded:
+            return 0
+        first = [pos // c * c for c in self.chunks]
+        if self.window is not None:
+            first.append(pos - self.window + 1)
+        return max(0, min(first))
+
+    def same_rows(self, other: "KVCacheSpec") -> bool:
+        """Whether both describe the same cached rows, whatever of them is in sight."""
+        return (self.num_kv_heads, self.head_dim, self.planes) == (other.num_kv_heads, other.head_dim, other.planes)
+
+    def covering(self, other: "KVCacheSpec") -> "KVCacheSpec":
+        """The same rows, kept for this spec's queries and the other's."""
+        if not (self.bounded and other.bounded):
+            return replace(self, window=None, chunks=())
+        windows = [w for w in (self.window, other.window) if w is not None]
+        return replace(self, window=max(windows, default=None), chunks=tuple(sorted(set(self.chunks) | set(other.chunks))))
 
 
 @dataclass(frozen=True)

@@ -44,7 +44,7 @@ class BiasedAttention(Part):
 
     def __init__(self, hidden_size: int, num_heads: int, num_kv_heads: int, key_dim: int, value_dim: int, scale: float,
                  slope_log2_span: float = 8.0, temp_coef: float = 0.0, temp_every: int = 0,
-                 value_mix: str | None = None, gate: bool = True) -> None:
+                 value_mix: str | None = None, gate: bool = True, maps: int = 1) -> None:
         if num_heads % num_kv_heads:
             raise ValueError(f"{num_heads} heads are not a multiple of {num_kv_heads} key/value heads")
         if key_dim > 256 or value_dim > 256:
@@ -55,9 +55,10 @@ class BiasedAttention(Part):
         self.key_dim, self.value_dim, self.scale = key_dim, value_dim, float(scale)
         self.slope_log2_span, self.temp_coef, self.temp_every = float(slope_log2_span), float(temp_coef), int(temp_every)
         self.value_mix, self.has_gate = value_mix, bool(gate)
-        self.v_at = -(-key_dim // 8) * 8
+        self.maps = maps  # query vectors a head and keys a key/value head
+        self.v_at = -(-maps * key_dim // 8) * 8
         self.row = -(-(self.v_at + value_dim) // 8) * 8
-        self.q_width, self.k_width = num_heads * key_dim, num_kv_heads * key_dim
+        self.q_width, self.k_width = num_heads * maps * key_dim, num_kv_heads * maps * key_dim
         self.v_width, self.out_width = num_kv_heads * value_dim, num_heads * value_dim
         self.out_padded = -(-self.out_width // 8) * 8
         self.proj_weight = self.out_weight = self.mix_weight = self.slopes = None
@@ -71,7 +72,7 @@ class BiasedAttention(Part):
         keeping at least two tiles; the parts are merged in their order by a second kernel."""
         if n_decode <= 0:
             return 1, False
-        blocks = n_decode * self.num_kv_heads * -(-(self.num_heads // self.num_kv_heads) // 32)
+        blocks = n_decode * self.num_kv_heads * -(-(self.num_heads // self.num_kv_heads) * self.maps // 32)
         tiles = max(1, -(-span // 32))
         return max(1, min(8 * K.sm_count() // blocks, tiles // 2, 32)), False
 

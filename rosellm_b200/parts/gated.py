@@ -1,4 +1,4 @@
-"""Gated feed-forward layers: dense, a mixture of experts, and a token-gated input.
+"""Gated feed-forward layers (and mixtures of ungated ones): dense, a mixture of experts, and a token-gated input.
 
 All three end in a product whose result goes to the residual stream or (``add=False``) to a
 buffer that the block normalises first.  The gate functions are those of csrc/gated_act.cuh:
@@ -66,13 +66,19 @@ class MixtureOfExperts(Part):
     """``num_experts`` gated feed-forward layers of which a token uses ``top``.
 
     Router logits ``z = W_router h`` with float32 accumulation and output; scores
-    ``s = softmax(z)`` over all experts, or (``score="sigmoid"``) each expert's ``sigmoid(z)``; the choice is made on ``s + correction`` (where the
+    ``s = softmax(z)`` over all experts, or (``score="sigmoid"``) each expert's ``sigmoid(z)``, or
+    (``score="chosen_softmax"``) ``s = z``, where the weights are the softmax over the chosen scores alone; the choice is made on ``s + correction`` (where the
     model has one), restricted, with groups, to the experts of the ``group_keep`` groups (of
     ``group_count`` equal groups of neighbours) whose best choice score is largest; the chosen
     experts' outputs are summed with their scores ``s`` as weights (not renormalised); with
     ``weight_input`` the weight multiplies the expert's input instead: the sum of ``expert(s * h)``.
     ``routing="table"``: no router; row ``token id`` of an integer table ``[vocab_size, top]`` (tensor ``table``; the
     entries of a row differ) names the token's experts, each with weight ``1 / top``.
+    ``gate`` may also name an activation of one input projection (``relu_squared``): an expert is then ``W_down act(W_up
+    h)`` and its tensor ``up_weight`` [experts * inner, hidden].
+    ``shared_inner`` > 0: a feed-forward of that inner size and of the same form (one input projection) runs for
+    every token and is added times ``sigmoid(W_sg h)``, one number a token (tensors ``shared_up_weight``,
+    ``shared_down_weight``, ``shared_gate_weight`` [1, hidden], the last in one product with the router).
     Routing, the experts' layout and their products all run on the device
     (csrc/moe.cu): a step's launches follow from its token count alone.
     Experts' tensors: ``gate_up_weight`` [experts * 2 * inner, hidden] (per expert the gate rows,
@@ -86,7 +92,7 @@ class MixtureOfExperts(Part):
     def __init__(self, hidden_size: int, inner_size: int, num_experts: int, top: int, group_count: int = 1,
                  group_keep: int = 1, gate: str = "silu", alpha: float = 1.0, limit: float = 0.0,
                  correction: bool = False, score: str = "softmax", weight_input: bool = False,
-                 routing: str = "router", vocab_size: int = 0) -> None:
+                 routing: str = "router", vocab_size: int = 0, shared_inner: int = 0) -> None:
         if routing not in ("router", "table"):
             raise ValueError(f"mixture of experts: routing {routing!r}; 'router' or 'table'")
         if routing == "table" and (vocab_size <= 0 or correction or group_count != 1):
@@ -112,14 +118,24 @@ class MixtureOfExperts(Part):
         self.hidden_size, self.inner_size = hidden_size, inner_size
         self.num_experts, self.top = num_experts, top
         self.group_count, self.group_keep = group_count, group_keep
-        self.gate, self.alpha, self.limit = _gate(gate), float(alpha), float(limit)
+        self.gated = gate not in K.UNITS
+        self.gate, self.alpha, self.limit = (_gate(gate) if self.gated else K.UNITS[gate]), float(alpha), float(limit)
+        self.shared_inner, self.shared_padded = int(shared_inner), -(-int(shared_inner) // 8) * 8
+        if shared_inner and (self.gated or routing != "router" or weight_input):
+            raise ValueError("mixture of experts: a shared feed-forward goes with experts of one input projection chosen by "
+                             "a router, whose outputs are weighted")
+        self.shared_act = K.ACTIVATIONS[gate] if shared_inner else None
         self.has_correction = bool(correction)
         self.router_weight = self.correction = self.gate_up_weight = self.down_weight = self.table = None
+        self.shared_up_weight = self.shared_down_weight = None
 
     def param_specs(self):
         E, f, hid = self.num_experts, self.inner_size, self.hidden_size
-        specs = [ParamSpec("gate_up_weight", (E * 2 * f, hid)),
+        specs = [ParamSpec("gate_up_weight", (E * 2 * f, hid)) if self.gated else ParamSpec("up_weight", (E * f, hid)),
                  ParamSpec("down_weight", (E * hid, f))]
+        if self.shared_inner:
+            specs += [ParamSpec("shared_up_weight", (self.shared_inner, hid)),
+                      ParamSpec("shared_down_weight", (hid, self.shared_inner)), ParamSpec("shared_gate_weight", (1, hid))]
         if self.routing == "table":
             specs.append(ParamSpec("table", (self.vocab_size, self.top), kind="int_table", below=E))
         else:
@@ -127,6 +143,21 @@ class MixtureOfExperts(Part):
         if self.has_correction:
             specs.append(ParamSpec("correction", (E,), kind="vector"))
         return specs
+
+    def bind(self, tensors) -> None:
+        t = dict(tensors)
+        if not self.gated:
+            t["gate_up_weight"] = t.pop("up_weight")
+        if self.shared_inner:
+            # the shared feed-forward's gate is one more row of the router; rows up to a multiple of 8 are zero
+            rows = [t["router_weight"], t.pop("shared_gate_weight")]
+            fill = -(self.num_experts + 1) % 8
+            t["router_weight"] = torch.nn.functional.pad(torch.cat(rows), (0, 0, 0, fill)).contiguous()
+            pad = self.shared_padded - self.shared_inner
+            if pad:  # units of zero weight: the activation maps 0 to 0
+                t["shared_up_weight"] = torch.nn.functional.pad(t["shared_up_weight"], (0, 0, 0, pad)).contiguous()
+                t["shared_down_weight"] = torch.nn.functional.pad(t["shared_down_weight"], (0, pad)).contiguous()
+        super().bind(t)
 
     def _table_route(self, ctx):
         """Routing by the table and its layout.  Both depend on the step's token ids alone, so a part that runs
@@ -159,34 +190,64 @@ class MixtureOfExperts(Part):
         got = routes[id(self)] = (weights, tiles, meta, row_token, place_of)
         return got
 
-    def forward(self, ctx, h, x, add: bool = True) -> None:
-        n, E, top, f, hid = ctx.n_tokens, self.num_experts, self.top, self.inner_size, self.hidden_size
+    def _route(self, ctx, h):
+        """Routing by the router: (weights, tiles, meta, row_token, place_of, weights by place or ``None``, the shared
+        feed-forward's gate logits or ``None``)."""
+        n, E, top = ctx.n_tokens, self.num_experts, self.top
         ws, i32 = ctx.workspace, torch.int32
-        by_place = None
+        ids = ws.get("moe_ids", (n * top,), i32)
+        weights = ws.get("moe_weights", (n * top,), torch.float32)
+        offsets = ws.get("moe_offsets", (E + 1,), i32)
+        tiles = ws.get("moe_tiles", (K.moe_max_tiles(n * top, E) * 3,), i32)
+        meta = ws.get("moe_meta", (4,), i32)
+        row_token = ws.get("moe_row_token", (n * top,), i32)
+        place_of = ws.get("moe_place_of", (n * top,), i32)
+        by_place = ws.get("moe_place_weight", (n * top,), torch.float32) if self.weight_input else None
+        full = ws.get("moe_logits", (n, self.router_weight.shape[0]), torch.float32)
+        K.linear(h, self.router_weight, None, full)
+        z = full[:, :E]
+        choice = dict(top=top, group_count=self.group_count, group_keep=self.group_keep, score=self.score, ids=ids,
+                      weights=weights)
+        if n <= K.MOE_ROUTE_MAX_TOKENS and n * top <= K.MOE_TABLE_ROUTE_MAX_PAIRS:
+            K.moe_select_route(z, self.correction, offsets=offsets, tiles=tiles, meta=meta, row_token=row_token,
+                               place_of=place_of, place_weight=by_place, **choice)
+        else:
+            counts = ws.get_zeroed("moe_counts", (E,), i32)
+            fill = ws.get_zeroed("moe_fill", (E,), i32)
+            K.moe_select(z, self.correction, counts=counts, **choice)
+            K.moe_plan(ids, counts, fill, offsets, tiles, meta, row_token, place_of, n_tokens=n, n_experts=E, top=top,
+                       weights=weights if self.weight_input else None, place_weight=by_place)
+        return weights, tiles, meta, row_token, place_of, by_place, full[:, E] if self.shared_inner else None
+
+    def _experts(self, ctx, h, x, add: bool):
+        """The experts' outputs, summed into ``x``, or (``x`` ``None``) left unsummed as a ``K.ExpertSum``."""
+        n, E, top, f, hid = ctx.n_tokens, self.num_experts, self.top, self.inner_size, self.hidden_size
+        ws = ctx.workspace
+        by_place = shared = shared_gate = None
         if self.routing == "table":
             weights, tiles, meta, row_token, place_of = self._table_route(ctx)
         else:
-            ids = ws.get("moe_ids", (n * top,), i32)
-            weights = ws.get("moe_weights", (n * top,), torch.float32)
-            counts = ws.get_zeroed("moe_counts", (E,), i32)
-            fill = ws.get_zeroed("moe_fill", (E,), i32)
-            z = ws.get("moe_logits", (n, E), torch.float32)
-            K.linear(h, self.router_weight, None, z)
-            K.moe_select(z, self.correction, top=top, group_count=self.group_count, group_keep=self.group_keep, ids=ids,
-                         weights=weights, counts=counts, score=self.score)
-            offsets = ws.get("moe_offsets", (E + 1,), i32)
-            tiles = ws.get("moe_tiles", (K.moe_max_tiles(n * top, E) * 3,), i32)
-            meta = ws.get("moe_meta", (4,), i32)
-            row_token = ws.get("moe_row_token", (n * top,), i32)
-            place_of = ws.get("moe_place_of", (n * top,), i32)
-            by_place = ws.get("moe_place_weight", (n * top,), torch.float32) if self.weight_input else None
-            K.moe_plan(ids, counts, fill, offsets, tiles, meta, row_token, place_of, n_tokens=n, n_experts=E, top=top,
-                       weights=weights if self.weight_input else None, place_weight=by_place)
+            weights, tiles, meta, row_token, place_of, by_place, shared_gate = self._route(ctx, h)
+        if self.weight_input:
+            weights = None
+        if self.shared_inner:
+            u = ws.get("moe_shared_inner", (n, self.shared_padded), ctx.act_dtype)
+            K.linear(h, self.shared_up_weight, None, u, act=self.shared_act)
+            shared = ws.get("moe_shared_out", (n, hid), torch.float32)
+            K.linear(u, self.shared_down_weight, None, shared)
         act = ws.get("moe_inner", (n * top, f), ctx.act_dtype)
         eo = ws.get("moe_expert_out", (n * top, hid), torch.float32)
-        K.moe_experts(h, self.gate_up_weight, self.down_weight, tiles, meta, row_token, place_of,
-                      None if self.weight_input else weights, act, eo, x, n_experts=E, top=top, ff=f, gate=self.gate,
-                      alpha=self.alpha, limit=self.limit, add=add, place_weight=by_place)
+        K.moe_experts(h, self.gate_up_weight, self.down_weight, tiles, meta, row_token, place_of, weights, act, eo, x,
+                      n_experts=E, top=top, ff=f, gate=self.gate, alpha=self.alpha, limit=self.limit, add=add,
+                      place_weight=by_place, shared=shared if x is not None else None, shared_gate=shared_gate)
+        return None if x is not None else K.ExpertSum(eo, weights, place_of, top, shared, shared_gate)
+
+    def forward(self, ctx, h, x, add: bool = True) -> None:
+        self._experts(ctx, h, x, add)
+
+    def forward_deferred(self, ctx, h) -> "K.ExpertSum":
+        """Everything but the sum of a token's experts, for a consumer that forms it itself."""
+        return self._experts(ctx, h, None, False)
 
 
 @register_part("feed_forward", "token_gated_input")

@@ -514,7 +514,8 @@ class CausalSelfAttention(Part):
 @register_part("feed_forward", "dense_mlp")
 class DenseMLP(Part):
     """``x += act(h W_in + b_in) W_out + b_out`` (rosellm/rosetrainer/model.py:331-349);
-    ``activation`` is ``gelu_tanh`` (model.py:274-277) or ``gelu_erf`` (``F.gelu``)."""
+    ``activation`` is ``gelu_tanh`` (model.py:274-277), ``gelu_erf`` (``F.gelu``) or ``relu_squared``
+    (max(u, 0)^2)."""
 
     graph_safe = True
     launches_replayable = True
@@ -523,7 +524,7 @@ class DenseMLP(Part):
     def __init__(self, hidden_size: int, inner_size: int, activation: str, bias: bool = True,
                  weights_in_out: bool = False) -> None:
         if activation not in K.ACTIVATIONS or activation == "none":
-            raise ValueError(f"activation {activation!r}; one of gelu_tanh, gelu_erf")
+            raise ValueError(f"activation {activation!r}; one of gelu_tanh, gelu_erf, relu_squared")
         self.hidden_size = hidden_size
         self.inner_size = inner_size
         self.activation = K.ACTIVATIONS[activation]
@@ -546,8 +547,8 @@ class DenseMLP(Part):
 
     def bind(self, tensors) -> None:
         """The products read rows in 16-byte pieces, so an inner size that is no multiple of 8
-        is filled up with units whose weights and bias are zero: their activation is 0 (both
-        GELU forms map 0 to 0) and they add nothing to the output."""
+        is filled up with units whose weights and bias are zero: their activation is 0 (every
+        activation maps 0 to 0) and they add nothing to the output."""
         super().bind(tensors)
         pad = -self.inner_size % 8
         self.inner_padded = self.inner_size + pad

@@ -1,4 +1,4 @@
-"""Softmax attention over the latest keys only, with normalised and rotated queries and keys, values of unit
+"""Softmax attention over the latest keys or the query's chunk only, with normalised and rotated queries and keys, values of unit
 root mean square and a temperature per head; optionally biases in the projections, a softmax sink (learned per
 head, or a constant) and an output gate (a logit per head, or per value column).
 
@@ -40,7 +40,10 @@ class WindowAttention(BiasedAttention):
     denominator, which has no key and no value and is not scaled; ``gate``: ``"head"`` (``W_g`` [heads, hidden]:
     head h's result times sigmoid((W_g h)_h)) or ``"element"`` (``W_g`` [heads * value_dim, hidden]: the merged
     heads times sigmoid(W_g h) element by element), read from the same input as the projections and packed
-    with them into one product."""
+    with them into one product; ``chunk``: a query at i sees only the keys j <= i with floor(j / chunk) =
+    floor(i / chunk), chunks counted from the sequence's first token (the cache gives a chunk's pages back once the
+    sequence has left it); ``own_kv=False``: the layer has queries alone and reads the keys and values of another
+    layer's cache (its runs carry ``cache_of``)."""
 
     takes_projection = True  # forward(.., proj=): the input times ``proj_weight``, made by the caller
 
@@ -48,9 +51,10 @@ class WindowAttention(BiasedAttention):
                  norm_eps: float, window: int | None = None, rot_dims: int = 0, rot_base: float = 10000.0,
                  qk_norm: bool = True, unit_values: bool = True, head_temperature: bool = True,
                  qk_norm_weights: bool = True, bias: bool = False, rot_scaling: dict | None = None,
-                 sink: "str | float | None" = None, gate: str | None = None) -> None:
+                 sink: "str | float | None" = None, gate: str | None = None, chunk: int | None = None,
+                 own_kv: bool = True, maps: int = 1) -> None:
         super().__init__(hidden_size, num_heads, num_kv_heads, key_dim, value_dim, scale, slope_log2_span=0.0,
-                         value_mix=None, gate=False)
+                         value_mix=None, gate=False, maps=maps)
         if gate not in (None, "head", "element"):
             raise ValueError(f"window attention: gate {gate!r}; None, 'head' or 'element'")
         if sink is not None and sink != "learned" and not isinstance(sink, (int, float)):
@@ -61,6 +65,11 @@ class WindowAttention(BiasedAttention):
         self.qk_norm_weights = bool(qk_norm_weights)
         if window is not None and window <= 0:
             raise ValueError(f"window attention: a window of {window} keys")
+        if chunk is not None and (chunk <= 0 or window is not None):
+            raise ValueError(f"window attention: chunks of {chunk} keys, and not beside a window")
+        if not own_kv and unit_values:
+            raise ValueError("window attention: a layer without values of its own cannot normalise them")
+        self.chunk, self.own_kv = None if chunk is None else int(chunk), bool(own_kv)
         if rot_dims < 0 or rot_dims % 2 or rot_dims > key_dim:
             raise ValueError(f"window attention: {rot_dims} turned entries of {key_dim}: an even count within the key size")
         self.window = None if window is None else int(window)
@@ -71,12 +80,15 @@ class WindowAttention(BiasedAttention):
         self.q_norm = self.k_norm = self.head_temp = self.sink = self.proj_bias = None
 
     def decode_plan_for(self, n_decode: int, span: int, act_dtype=None) -> tuple[int, bool]:
-        return super().decode_plan_for(n_decode, span if self.window is None else min(span, self.window), act_dtype)
+        for most in (self.window, self.chunk):
+            span = span if most is None else min(span, most)
+        return super().decode_plan_for(n_decode, span, act_dtype)
 
     def param_specs(self):
         hid = self.hidden_size
-        specs = [ParamSpec("q_weight", (self.q_width, hid)), ParamSpec("k_weight", (self.k_width, hid)),
-                 ParamSpec("v_weight", (self.v_width, hid)), ParamSpec("out_weight", (hid, self.out_width))]
+        specs = [ParamSpec("q_weight", (self.q_width, hid)), ParamSpec("out_weight", (hid, self.out_width))]
+        if self.own_kv:
+            specs[1:1] = [ParamSpec("k_weight", (self.k_width, hid)), ParamSpec("v_weight", (self.v_width, hid))]
         if self.qk_norm and self.qk_norm_weights:
             specs += [ParamSpec("q_norm", (self.key_dim,), kind="vector", init="ones"),
                       ParamSpec("k_norm", (self.key_dim,), kind="vector", init="ones")]
@@ -93,17 +105,18 @@ class WindowAttention(BiasedAttention):
         return specs
 
     def cache_spec(self):
-        return KVCacheSpec(self.num_kv_heads, self.row, self.window, planes=1)
+        return KVCacheSpec(self.num_kv_heads, self.row, self.window, planes=1,
+                           chunks=() if self.chunk is None else (self.chunk,))
 
     def bind(self, tensors) -> None:
         t = dict(tensors)
-        parts = [t["q_weight"], t["k_weight"], t["v_weight"]] + ([t["gate_weight"]] if self.has_gate else [])
-        self.proj_weight, offs = pack_rows(parts)
-        self.offsets = dict(zip(("q", "k", "v", "g"), offs))
+        roles = ["q"] + (["k", "v"] if self.own_kv else []) + (["gate"] if self.has_gate else [])
+        self.proj_weight, offs = pack_rows([t[f"{r}_weight"] for r in roles])
+        self.offsets = dict(zip((r[0] for r in roles), offs))
         self.proj_bias = None
         if self.has_bias:  # the packed product's bias: the three biases at their rows, zero elsewhere
             self.proj_bias = torch.zeros(self.proj_weight.shape[0], dtype=torch.float32, device=self.proj_weight.device)
-            for name, role in (("q", "q_bias"), ("k", "k_bias"), ("v", "v_bias")):
+            for name, role in ((r, f"{r}_bias") for r in roles if r != "gate"):
                 self.proj_bias[self.offsets[name]:self.offsets[name] + t[role].numel()] = t[role]
         self.sink = t.get("sink")
         if self.sink_kind is not None and self.sink_kind != "learned":
@@ -115,6 +128,10 @@ class WindowAttention(BiasedAttention):
         self.q_norm, self.k_norm, self.head_temp = t.get("q_norm"), t.get("k_norm"), t.get("head_temp")
         self.slopes = self.mix_weight = None
 
+    def _attention_options(self) -> dict:
+        """What a kind of attention built on this one hands the attention kernel beyond the common arguments."""
+        return {}
+
     def forward(self, ctx, run, h, x, add: bool = True, proj=None) -> None:
         n, ws = ctx.n_tokens, ctx.workspace
         if proj is None:  # else: a block has multiplied this part's packed weight together with others'
@@ -124,8 +141,12 @@ class WindowAttention(BiasedAttention):
             raise ValueError("window attention: a projection made by the block carries no biases")
         o = self.offsets
         q = proj[:, o["q"]:o["q"] + self.q_width]
-        k = proj[:, o["k"]:o["k"] + self.k_width]
-        v = proj[:, o["v"]:o["v"] + self.v_width]
+        k = v = None
+        if self.own_kv:
+            k = proj[:, o["k"]:o["k"] + self.k_width]
+            v = proj[:, o["v"]:o["v"] + self.v_width]
+        elif run.writes_cache:
+            raise ValueError("window attention: a layer without keys and values of its own reads another layer's cache")
         gate = proj[:, o["g"]:o["g"] + self.gate_width] if self.has_gate else None
         pool, table = ctx.kv_pool(run.cache_key), ctx.block_table(run.cache_key)
         stored = False
@@ -137,7 +158,8 @@ class WindowAttention(BiasedAttention):
                               dv=self.value_dim, eps=self.norm_eps, q_norm=self.q_norm, k_norm=self.k_norm,
                               freq=self.rotary.frequencies(ctx.device) if self.rotary is not None else None,
                               rot_dims=self.rot_dims, unit_values=self.unit_values,
-                              unit_qk=self.qk_norm and not self.qk_norm_weights, cache=target)
+                              unit_qk=self.qk_norm and not self.qk_norm_weights, cache=target, maps=self.maps,
+                              rot_mult=self.rotary.mult if self.rotary is not None else 1.0)
         if run.writes_cache and not stored:
             K.bias_kv_store(k, v, pool, table, ctx.positions, ctx.req_of_token, ctx.slots, v_at=self.v_at,
                             max_pos=ctx.cache.max_seq_len)
@@ -147,14 +169,14 @@ class WindowAttention(BiasedAttention):
         else:  # the fill stays zero: see the state mixers' output buffer
             buf = ws.get_zeroed(f"biased_attn_out_{self.out_width}_{self.out_padded}", (n, self.out_padded), ctx.act_dtype)
             out = buf[:, :self.out_width]
-        mma = K.bias_attention_tensor_cores(ctx.act_dtype, self.key_dim, self.value_dim)
+        mma = K.bias_attention_tensor_cores(ctx.act_dtype, self.key_dim, self.value_dim, self.maps)
         if self._shape is None or self._shape[0] != mma:
-            self._shape = (mma, K.bias_attention_shape(self.num_heads // self.num_kv_heads, mma)[1])
+            self._shape = (mma, K.bias_attention_shape(self.num_heads // self.num_kv_heads, mma, self.maps)[1])
         wide = self._shape[1] > 16  # the tokens a block takes must divide the tiles the step is cut into
         splits = step_decode_plan(self, ctx)[0]
         part_o = part_ml = None
         if splits > 1:
-            rows = ctx.n_decode * self.num_heads * splits
+            rows = ctx.n_decode * self.num_heads * self.maps * splits
             part_o = ws.get("biased_attn_part_o", (rows, self.value_dim), torch.float32)
             part_ml = ws.get("biased_attn_part_ml", (rows, 2), torch.float32)
         K.bias_attention(q, gate, pool, table, ctx.q_start, ctx.kv_len, ctx.slots, out, n_heads=self.num_heads,
@@ -163,5 +185,6 @@ class WindowAttention(BiasedAttention):
                          tile_tokens=64 if wide else 16, decode_reqs=ctx.decode_reqs, n_decode=ctx.n_decode,
                          max_pos=ctx.cache.max_seq_len, n_splits=splits, part_o=part_o, part_ml=part_ml, tensor_cores=mma,
                          window=self.window or 0, head_scale=self.head_temp, sink=self.sink,
-                         gate_per_head=self.gate_kind == "head")
+                         gate_per_head=self.gate_kind == "head", chunk=self.chunk or 0, maps=self.maps,
+                         **self._attention_options())
         K.linear(buf, self.out_weight, None, x, residual=add)
