@@ -67,6 +67,10 @@ def parse_args():
                         "share one norm; attention over a window with a sink, rotary attention with a gate per head, latent "
                         "attention with a query latent; experts named by a table; a stretch of layers run twice) beside "
                         "Lebedra, the nearest shipped design, at equal width, runs of layers and vocabulary, random weights")
+    p.add_argument("--compare-vebotar", action="store_true",
+                   help="instead of the default workload: prefill and decode of the Vebotar design (differential attention "
+                        "over chunks, a stream of two copies, routed experts beside a shared one) and of Soporax's windowed "
+                        "attention and experts at equal width, depth and vocabulary")
     p.add_argument("--compare-lebedra", action="store_true",
                    help="instead of the default workload: prefill and decode of the Lebedra design (latent attention, "
                         "mixture of experts) beside GPT-2 of equal width, depth and vocabulary, at layer sizes of "
@@ -880,6 +884,81 @@ def compare_soporax(args):
     return 0
 
 
+# Layer sizes for --compare-vebotar: width; heads, key/value heads, size of a query or key vector of one map, value size
+# and the chunks' size; experts, experts a token, their inner size and the shared expert's; and of the Soporax arm:
+# heads, key/value heads, key and value size and window of its attention (projections of the same sizes), and the inner
+# size of its gated experts (three matrices where Vebotar's have two: as many weights an expert).
+VEBOTAR_SIZES = {
+    "1024": dict(width=1024, heads=8, kv_heads=2, dim=64, vdim=128, chunk=256, experts=16, top=2, expert_ff=1536, shared_ff=1536,
+                 s_heads=16, s_kv_heads=4, s_dim=64, s_vdim=64, s_expert_ff=1024),
+    "2048": dict(width=2048, heads=16, kv_heads=4, dim=64, vdim=128, chunk=256, experts=32, top=4, expert_ff=2112, shared_ff=2112,
+                 s_heads=16, s_kv_heads=4, s_dim=128, s_vdim=128, s_expert_ff=1408),
+}
+
+
+def vebotar_config(z: dict, layers: int, vocab: int, positions: int):
+    """Every third layer reads the keys and values of the layer before it."""
+    from rosellm_b200.config.vebotar import VebotarConfig
+
+    attn = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["vdim"], "scale": z["dim"] ** -0.5,
+            "diff": 0.3, "mask": {"size": z["chunk"]},
+            "rot": {"dims": z["dim"], "base": 500000.0, "scaling": {"factor": 8.0, "original": 256, "fast": 16.0, "slow": 2.0}}}
+    moe = {"kind": "moe", "expert": {"ff": z["expert_ff"]}, "router": {"experts": z["experts"], "top": z["top"]},
+           "shared": {"ff": z["shared_ff"]}}
+    return VebotarConfig.from_dict({
+        "architecture": "Vebotar", "vocab": vocab, "width": z["width"], "max_positions": positions, "norm": {"eps": 1e-5},
+        "embedding": {"scale": float(z["width"]) ** 0.5}, "streams": 2,
+        "layers": [{"type": "attention", "mixer": dict(attn, kv_from=i - 1) if i % 3 == 2 else attn, "mlp": moe}
+                   for i in range(layers)]})
+
+
+def vebotar_neighbour_config(z: dict, layers: int, vocab: int, positions: int):
+    """Soporax with windowed attention and experts in every layer."""
+    from rosellm_b200.config.soporax import SoporaxConfig
+
+    attn = {"heads": z["s_heads"], "kv_heads": z["s_kv_heads"], "dim": z["s_dim"], "vdim": z["s_vdim"], "scale": z["s_dim"] ** -0.5,
+            "mask": {"size": z["chunk"]}}
+    moe = {"kind": "moe", "expert": {"ff": z["s_expert_ff"]}, "router": {"experts": z["experts"], "top": z["top"]}}
+    return SoporaxConfig.from_dict({
+        "architecture": "Soporax", "vocab": vocab, "width": z["width"], "max_positions": positions, "norm": {"eps": 1e-5},
+        "logit_scale": 0.5, "layers": [{"type": "attention", "mixer": attn, "mlp": moe} for _ in range(layers)]})
+
+
+def compare_vebotar(args):
+    """Prefill (2 x 1024 tokens) and decode (batch 8 and 64, 512 cached tokens) of Vebotar and of Soporax (the nearest
+    shipped design, here with windowed attention and experts in all layers) at equal width, depth, vocabulary,
+    projection sizes and weights an expert: device time by CUDA events, as the default workload."""
+    layers, vocab, positions = 6, 32000, 1024
+    clocks = Clocks()
+    clocks.start()
+    out = {"metric": "prefill and decode of Vebotar beside Soporax at equal width", "unit": "tokens/s", "n_gpus": 1,
+           "steps": args.steps, "warmup": args.warmup, "dtype": "bf16" if args.dtype == "bfloat16" else "fp32",
+           "data": "synthetic (random token ids, random weights)", "layers": layers, "vocab": vocab, "sizes": {}}
+    for name, z in VEBOTAR_SIZES.items():
+        row = {}
+        for label, cfg in (("vebotar", vebotar_config(z, layers, vocab, positions)),
+                           ("soporax", vebotar_neighbour_config(z, layers, vocab, positions))):
+            h = Harness(cfg, args.dtype, 64, graphs=not args.no_graphs)
+            try:
+                pms = h.prefill()
+                rec = {"prefill_2x1024_ms": round(pms, 4), "prefill_tok_s": round(2048 / (pms * 1e-3), 1),
+                       "weight_mb": round(h.runner.model.weight_bytes() / 1e6, 1)}
+                for b in (8, 64):
+                    ms, launches, gms, _ = h.device_decode(b, args.context, max(16, args.steps // 2), max(4, args.warmup // 2))
+                    rec[f"decode_b{b}_ms"] = round(ms, 4)
+                    rec[f"decode_b{b}_tok_s"] = round(b / (ms * 1e-3), 1)
+                    rec[f"decode_b{b}_launches"] = launches
+                    if gms is not None:
+                        rec[f"decode_b{b}_graph_ms"] = round(gms, 4)
+                row[label] = rec
+            finally:
+                h.close()
+        out["sizes"][name] = row
+    out["clocks"] = clocks.stop()
+    print(json.dumps(out))
+    return 0
+
+
 def main():
     args = parse_args()
     if args.gpus != 1:
@@ -893,6 +972,8 @@ def main():
         return compare_fikevik(args)
     if args.compare_soporax:
         return compare_soporax(args)
+    if args.compare_vebotar:
+        return compare_vebotar(args)
     if args.impl == "reference":
         run_reference(args)
     else:

@@ -91,7 +91,7 @@ class ParamSpec:
     shape: tuple[int, ...]
     kind: str = "matrix"
     transpose: bool = False
-    # how the random-weights mode fills it: "normal" or "ones" (a norm's scale)
+    # how the random-weights mode fills it: "normal", "ones" (a norm's scale), "zeros" or "eye" (a square mixing matrix)
     init: str = "normal"
     # an integer table's entries lie in [0, below); the random-weights mode draws every row's entries distinct
     below: int = 0

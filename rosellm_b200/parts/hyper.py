@@ -26,8 +26,9 @@ class HyperConnection(Part):
         self.in_weight = self.out_weight = self.mix = None
 
     def param_specs(self):
-        return [ParamSpec("in_weight", (self.copies,), kind="vector"), ParamSpec("out_weight", (self.copies,), kind="vector"),
-                ParamSpec("mix", (self.copies, self.copies), kind="vector")]
+        return [ParamSpec("in_weight", (self.copies,), kind="vector", init="ones"),
+                ParamSpec("out_weight", (self.copies,), kind="vector", init="ones"),
+                ParamSpec("mix", (self.copies, self.copies), kind="vector", init="eye")]
 
 
 @register_part("block", "hyper_connections")

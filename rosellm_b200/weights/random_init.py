@@ -62,6 +62,8 @@ def random_tensors(
             noise = torch.randn(shape, generator=g, dtype=torch.float32) * std
             if p.spec.init == "ones":
                 t = torch.ones(shape) + (noise if norm_affine == "random" else 0.0)
+            elif p.spec.init == "eye":
+                t = torch.eye(*shape) + (noise if norm_affine == "random" else 0.0)
             elif p.spec.init == "zeros":
                 t = noise if norm_affine == "random" else torch.zeros(shape)
             else:
