@@ -885,13 +885,13 @@ def compare_soporax(args):
 
 
 # Layer sizes for --compare-vebotar: width; heads, key/value heads, size of a query or key vector of one map, value size
-# and the chunks' size; experts, experts a token, their inner size and the shared expert's; and of the Soporax arm:
+# and the chunks' size (both arms see all earlier keys of a prompt and of a decoded token); experts, experts a token, their inner size and the shared expert's; and of the Soporax arm:
 # heads, key/value heads, key and value size and window of its attention (projections of the same sizes), and the inner
 # size of its gated experts (three matrices where Vebotar's have two: as many weights an expert).
 VEBOTAR_SIZES = {
-    "1024": dict(width=1024, heads=8, kv_heads=2, dim=64, vdim=128, chunk=256, experts=16, top=2, expert_ff=1536, shared_ff=1536,
+    "1024": dict(width=1024, heads=8, kv_heads=2, dim=64, vdim=128, chunk=1024, experts=16, top=2, expert_ff=1536, shared_ff=1536,
                  s_heads=16, s_kv_heads=4, s_dim=64, s_vdim=64, s_expert_ff=1024),
-    "2048": dict(width=2048, heads=16, kv_heads=4, dim=64, vdim=128, chunk=256, experts=32, top=4, expert_ff=2112, shared_ff=2112,
+    "2048": dict(width=2048, heads=16, kv_heads=4, dim=64, vdim=128, chunk=1024, experts=32, top=4, expert_ff=2112, shared_ff=2112,
                  s_heads=16, s_kv_heads=4, s_dim=128, s_vdim=128, s_expert_ff=1408),
 }
 

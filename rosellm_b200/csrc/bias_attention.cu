@@ -30,7 +30,8 @@
 // `bias_attn_kernel`: rows of a block are (token, head) pairs that share a key/value head, so a key tile
 // fetched once serves all of a group's heads; 32 rows x 32 keys a round, online softmax, float32 on the CUDA
 // cores.  A decoded token is a tile of one token; where a step has few of them, the keys of each are cut into
-// parts, a block a part, and `bias_attn_merge_kernel` puts the parts together in their order.
+// parts, a block a part, and `bias_attn_merge_kernel` puts the parts together in their order.  Queries, keys and
+// probabilities are read from shared memory 16 bytes at a time.
 #include <math_constants.h>
 
 #include "common.cuh"
@@ -38,6 +39,11 @@
 namespace rl {
 
 constexpr int BA_ROWS = 32, BA_KEYS = 32, BA_THREADS = 128;  // BA_ROWS: the rows of a prompt tile's block
+constexpr int BA_LDP = BA_KEYS + 4;                           // row stride of the probabilities in shared memory
+
+__host__ __device__ __forceinline__ int bias_up4(int n) { return (n + 3) & ~3; }
+// the next odd multiple of 4 from n on (n a multiple of 4)
+__host__ __device__ __forceinline__ int bias_row4(int n) { return n | 4; }
 
 struct BiasAttnParams {
   const float* q;  // [tokens, ldq]; head h at columns [h * dk, (h + 1) * dk)
@@ -92,7 +98,7 @@ namespace rl {
 
 // LPR lanes share a row (their keys tx + LPR b, their value columns tx + LPR c), RPT rows a thread: a block has
 // (BA_THREADS / LPR) * RPT rows.  Prompt tiles run 8 lanes x 2 rows (32 rows); a decoded token has only its
-// group's heads as rows, so its blocks run 16 or 32 lanes a row (8 or 4 rows) and every thread has work.
+// group's heads as rows, so its blocks run 32 lanes a row (4 rows, or 8 with two a thread) and every thread has work.
 // With two maps the first half of the rows are (token, head) pairs of map 1, the second half the same pairs of map 2.
 template <typename T, int LPR, int RPT, int DVC, typename TOut, int MAPS>
 __global__ __launch_bounds__(BA_THREADS) void bias_attn_kernel(const BiasAttnParams p) {
@@ -125,11 +131,13 @@ __global__ __launch_bounds__(BA_THREADS) void bias_attn_kernel(const BiasAttnPar
   const int HB = p.heads_per_block;
   const int dk = p.dk, dv = p.dv;
   const int kd = MAPS * dk;  // a token's keys
-  const int ldq_s = dk | 1, ldk_s = kd | 1, ldv_s = LPR * DVC;
+  // In shared memory a vector of dk entries is filled up to dk4 with zeros and read 16 bytes at a time; row strides are
+  // odd multiples of 16 bytes, so that eight rows at one entry lie in different banks.
+  const int dk4 = bias_up4(dk), ldq_s = bias_row4(dk4), ldk_s = bias_row4(MAPS * dk4), ldv_s = LPR * DVC;
   float* Qs = ba_s;                        // [ROWS][ldq_s]
   float* Ks = Qs + ROWS * ldq_s;           // [BA_KEYS][ldk_s]
   float* Vs = Ks + BA_KEYS * ldk_s;        // [BA_KEYS][ldv_s]
-  float* Ps = Vs + BA_KEYS * ldv_s;        // [ROWS][BA_KEYS + 1]
+  float* Ps = Vs + BA_KEYS * ldv_s;        // [ROWS][BA_LDP]
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int ty = tid / LPR, tx = tid % LPR;
   // queries
@@ -137,7 +145,7 @@ __global__ __launch_bounds__(BA_THREADS) void bias_attn_kernel(const BiasAttnPar
     const int pr = r % PAIRS, tl = pr / HB, hl = pr - tl * HB;
     const bool ok = tl < n_tok && hb0 + hl < hg;
     const float* src = p.q + (size_t)(t_begin + first + tl) * p.ldq + (size_t)(g * hg + hb0 + hl) * kd + (r / PAIRS) * dk;
-    for (int d = lane; d < dk; d += 32) Qs[r * ldq_s + d] = ok ? src[d] : 0.f;
+    for (int d = lane; d < dk4; d += 32) Qs[r * ldq_s + d] = ok && d < dk ? src[d] : 0.f;
   }
   int row_pos[RPT], row_lo[RPT], row_head[RPT];
   float row_mul[RPT], row_slope[RPT], m[RPT], l[RPT];
@@ -185,9 +193,11 @@ __global__ __launch_bounds__(BA_THREADS) void bias_attn_kernel(const BiasAttnPar
     }
   };
   constexpr int EV = 16 / (int)sizeof(T);  // elements of a 16-byte piece
-  const bool vec = kd % EV == 0 && dv % EV == 0 && p.row % EV == 0 && p.v_at % EV == 0 &&
+  const bool vec = dk % 4 == 0 && kd % EV == 0 && dv % EV == 0 && p.row % EV == 0 && p.v_at % EV == 0 &&
                    (reinterpret_cast<uintptr_t>(p.pool) & 15) == 0;
-  for (int i = tid; i < BA_KEYS * ldv_s; i += BA_THREADS) Vs[i] = 0.f;  // the fill beyond dv stays zero
+  // the fill beyond dk and dv stays zero
+  for (int i = tid; i < BA_KEYS * ldk_s; i += BA_THREADS) Ks[i] = 0.f;
+  for (int i = tid; i < BA_KEYS * ldv_s; i += BA_THREADS) Vs[i] = 0.f;
   int j_begin = first_seen / BA_KEYS * BA_KEYS, j_end = last_pos + 1;  // the keys this block walks
   if (parted) {
     const int tiles_all = (last_pos + BA_KEYS) / BA_KEYS - j_begin / BA_KEYS;
@@ -210,9 +220,10 @@ __global__ __launch_bounds__(BA_THREADS) void bias_attn_kernel(const BiasAttnPar
         uint4 raw = make_uint4(0u, 0u, 0u, 0u);
         if (src != nullptr) raw = *reinterpret_cast<const uint4*>(src + (is_v ? p.v_at : 0) + at);
         const T* e = reinterpret_cast<const T*>(&raw);
-        float* dst = is_v ? Vs + jj * ldv_s + at : Ks + jj * ldk_s + at;
+        float* dst = is_v ? Vs + jj * ldv_s + at : Ks + jj * ldk_s + at;  // dk4 = dk here: a token's keys are one run
 #pragma unroll
-        for (int x = 0; x < EV; ++x) dst[x] = to_f32(e[x]);
+        for (int x = 0; x < EV; x += 4)
+          *reinterpret_cast<float4*>(dst + x) = make_float4(to_f32(e[x]), to_f32(e[x + 1]), to_f32(e[x + 2]), to_f32(e[x + 3]));
       }
     } else {
       const int per_key = kd + dv;
@@ -223,24 +234,25 @@ __global__ __launch_bounds__(BA_THREADS) void bias_attn_kernel(const BiasAttnPar
         const bool is_v = c >= kd;
         const float val = src != nullptr ? to_f32(src[is_v ? p.v_at + c - kd : c]) : 0.f;
         if (is_v) Vs[jj * ldv_s + c - kd] = val;
-        else Ks[jj * ldk_s + c] = val;
+        else Ks[jj * ldk_s + (MAPS == 2 && c >= dk ? dk4 + c - dk : c)] = val;
       }
     }
     locate(j0 + BA_KEYS, buf ^ 1);
     __syncthreads();
     float s[RPT][KPT] = {};
     const float* q0 = Qs + (ty * RPT) * ldq_s;
-    const float* kb = Ks + tx * ldk_s + map * dk;
-#pragma unroll 4
-    for (int d = 0; d < dk; ++d) {
-      float qa[RPT];
+    const float* kb = Ks + tx * ldk_s + map * dk4;
+#pragma unroll 2
+    for (int d = 0; d < dk4; d += 4) {
+      float4 qa[RPT];
 #pragma unroll
-      for (int a = 0; a < RPT; ++a) qa[a] = q0[a * ldq_s + d];
+      for (int a = 0; a < RPT; ++a) qa[a] = *reinterpret_cast<const float4*>(q0 + a * ldq_s + d);
 #pragma unroll
       for (int b = 0; b < KPT; ++b) {
-        const float kv = kb[b * LPR * ldk_s + d];
+        const float4 kv = *reinterpret_cast<const float4*>(kb + b * LPR * ldk_s + d);
 #pragma unroll
-        for (int a = 0; a < RPT; ++a) s[a][b] = fmaf(qa[a], kv, s[a][b]);
+        for (int a = 0; a < RPT; ++a)
+          s[a][b] = fmaf(qa[a].w, kv.w, fmaf(qa[a].z, kv.z, fmaf(qa[a].y, kv.y, fmaf(qa[a].x, kv.x, s[a][b]))));
       }
     }
 #pragma unroll
@@ -261,7 +273,7 @@ __global__ __launch_bounds__(BA_THREADS) void bias_attn_kernel(const BiasAttnPar
 #pragma unroll
       for (int b = 0; b < KPT; ++b) {
         const float pr = s[a][b] == -CUDART_INF_F ? 0.f : expf(s[a][b] - m_new);
-        Ps[(ty * RPT + a) * (BA_KEYS + 1) + tx + LPR * b] = pr;
+        Ps[(ty * RPT + a) * BA_LDP + tx + LPR * b] = pr;
         sum += pr;
       }
 #pragma unroll
@@ -272,18 +284,21 @@ __global__ __launch_bounds__(BA_THREADS) void bias_attn_kernel(const BiasAttnPar
       for (int c = 0; c < DVC; ++c) acc[a][c] *= corr;
     }
     __syncwarp();  // a row's probabilities are written and read by the lanes of one warp
-    const float* p0 = Ps + (ty * RPT) * (BA_KEYS + 1);
-#pragma unroll 4
-    for (int jj = 0; jj < BA_KEYS; ++jj) {
-      float w[RPT];
+    const float* p0 = Ps + (ty * RPT) * BA_LDP;
+#pragma unroll 2
+    for (int j4 = 0; j4 < BA_KEYS; j4 += 4) {
+      float w[RPT][4];
 #pragma unroll
-      for (int a = 0; a < RPT; ++a) w[a] = p0[a * (BA_KEYS + 1) + jj];
-      const float* vr = Vs + jj * ldv_s + tx;
+      for (int a = 0; a < RPT; ++a) *reinterpret_cast<float4*>(w[a]) = *reinterpret_cast<const float4*>(p0 + a * BA_LDP + j4);
 #pragma unroll
-      for (int c = 0; c < DVC; ++c) {
-        const float v = vr[LPR * c];
+      for (int jj = 0; jj < 4; ++jj) {
+        const float* vr = Vs + (j4 + jj) * ldv_s + tx;
 #pragma unroll
-        for (int a = 0; a < RPT; ++a) acc[a][c] = fmaf(w[a], v, acc[a][c]);
+        for (int c = 0; c < DVC; ++c) {
+          const float v = vr[LPR * c];
+#pragma unroll
+          for (int a = 0; a < RPT; ++a) acc[a][c] = fmaf(w[a][jj], v, acc[a][c]);
+        }
       }
     }
   }
@@ -395,51 +410,52 @@ __global__ __launch_bounds__(128) void bias_attn_merge_kernel(const BiasAttnPara
   }
 }
 
-// The same for two maps: a warp a (decoded request, head) puts each map's parts together, then forms the difference and
-// brings it to unit root mean square.  dv <= 256: eight columns a lane.
+// The same for two maps: a block a (decoded request, head), a thread two columns (dv <= 256), which puts each map's parts
+// together, forms the difference and brings it to unit root mean square.
 template <typename TOut>
 __global__ __launch_bounds__(128) void bias_attn_merge_maps_kernel(const BiasAttnParams p) {
+  __shared__ float part_w[2][32];  // a part's weight over its map's sum; the second map's times -lambda
+  __shared__ float scratch[33];
   pdl_begin();
-  const int dec = blockIdx.x, req = p.decode_reqs[dec];
+  const int dec = blockIdx.x, head = blockIdx.y, req = p.decode_reqs[dec];
   if (p.slots[req] < 0) return;
-  const int tok = p.q_start[req], dv = p.dv;
+  const int dv = p.dv, n = p.n_splits;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const int head = blockIdx.y * 4 + warp;
-  if (head >= p.n_heads) return;
-  float r[8];
-#pragma unroll
-  for (int c = 0; c < 8; ++c) r[c] = 0.f;
-  const float lambda = *p.diff_lambda;
-#pragma unroll
-  for (int map = 0; map < 2; ++map) {
-    const size_t at = (((size_t)dec * p.n_heads + head) * 2 + map) * p.n_splits;
-    const float ms = lane < p.n_splits ? p.part_ml[2 * (at + lane)] : -CUDART_INF_F;
-    const float ls = lane < p.n_splits ? p.part_ml[2 * (at + lane) + 1] : 0.f;
+  const size_t at = ((size_t)dec * p.n_heads + head) * 2 * n;
+  if (warp < 2) {
+    const float ms = lane < n ? p.part_ml[2 * (at + warp * n + lane)] : -CUDART_INF_F;
+    const float ls = lane < n ? p.part_ml[2 * (at + warp * n + lane) + 1] : 0.f;
     const float M = warp_max(ms);
     const float w = ms == -CUDART_INF_F ? 0.f : expf(ms - M);
     float L = 0.f;
-    for (int s = 0; s < p.n_splits; ++s) L = fmaf(__shfl_sync(0xffffffffu, ls, s), __shfl_sync(0xffffffffu, w, s), L);
-    const float factor = (map == 0 ? 1.0f : -lambda) / L;
-#pragma unroll
-    for (int c = 0; c < 8; ++c) {
-      const int col = c * 32 + lane;
-      if (c * 32 >= dv) break;
-      float acc = 0.f;
-      for (int s = 0; s < p.n_splits; ++s) {
-        const float ws = __shfl_sync(0xffffffffu, w, s);
-        if (col < dv && ws != 0.f) acc = fmaf(p.part_o[(at + s) * dv + col], ws, acc);
-      }
-      r[c] = fmaf(acc, factor, r[c]);
-    }
+    for (int s = 0; s < n; ++s) L = fmaf(__shfl_sync(0xffffffffu, ls, s), __shfl_sync(0xffffffffu, w, s), L);
+    part_w[warp][lane] = w * ((warp == 0 ? 1.0f : -*p.diff_lambda) / L);
   }
-  float ss = 0.f;
+  __syncthreads();
+  float r[2] = {0.f, 0.f}, ss = 0.f;
 #pragma unroll
-  for (int c = 0; c < 8; ++c) ss = fmaf(r[c], r[c], ss);
-  const float mul = p.diff_mul / sqrtf(warp_sum(ss) / (float)dv + p.diff_eps);
-  TOut* o = reinterpret_cast<TOut*>(p.out) + (size_t)tok * p.ldo + (size_t)head * dv;
+  for (int c = 0; c < 2; ++c) {
+    const int col = threadIdx.x + 128 * c;
+    if (col < dv) {
 #pragma unroll
-  for (int c = 0; c < 8; ++c)
-    if (c * 32 + lane < dv) o[c * 32 + lane] = from_f32<TOut>(r[c] * mul);
+      for (int map = 0; map < 2; ++map) {
+        const float* o = p.part_o + (at + (size_t)map * n) * dv + col;
+        float acc = 0.f;
+#pragma unroll 4
+        for (int s = 0; s < n; ++s) {
+          const float w = part_w[map][s], v = o[(size_t)s * dv];
+          acc = fmaf(w != 0.f ? v : 0.f, w, acc);  // a part without keys counts nothing, whatever lies there
+        }
+        r[c] += acc;
+      }
+    }
+    ss = fmaf(r[c], r[c], ss);
+  }
+  const float mul = p.diff_mul / sqrtf(block_sum(ss, scratch) / (float)dv + p.diff_eps);
+  TOut* out = reinterpret_cast<TOut*>(p.out) + (size_t)p.q_start[req] * p.ldo + (size_t)head * dv;
+#pragma unroll
+  for (int c = 0; c < 2; ++c)
+    if (threadIdx.x + 128 * c < dv) out[threadIdx.x + 128 * c] = from_f32<TOut>(r[c] * mul);
 }
 
 // mix: 0 values as they are; 1 also left in v_src (this layer is the source); 2 mixed with v_src by *lambda.
@@ -480,8 +496,9 @@ __global__ void bias_kv_store_kernel(const float* __restrict__ k, long ldk, cons
 template <typename T, int LPR, int RPT, int DVC, typename TOut, int MAPS>
 static void launch_bias_attn(const BiasAttnParams& p, dim3 grid, cudaStream_t stream) {
   constexpr int ROWS = BA_THREADS / LPR * RPT;
-  const size_t smem = ((size_t)ROWS * (p.dk | 1) + (size_t)BA_KEYS * (MAPS * p.dk | 1) + (size_t)BA_KEYS * LPR * DVC +
-                       (size_t)ROWS * (BA_KEYS + 1)) * sizeof(float);
+  const int dk4 = bias_up4(p.dk);
+  const size_t smem = ((size_t)ROWS * bias_row4(dk4) + (size_t)BA_KEYS * bias_row4(MAPS * dk4) + (size_t)BA_KEYS * LPR * DVC +
+                       (size_t)ROWS * BA_LDP) * sizeof(float);
   auto kernel = bias_attn_kernel<T, LPR, RPT, DVC, TOut, MAPS>;
   if (smem > 48 * 1024) {
     static bool raised = false;
@@ -498,12 +515,12 @@ template <typename T, typename TOut, int MAPS>
 static void dispatch_bias_attn(const BiasAttnParams& p, int rows, dim3 grid, cudaStream_t stream) {
   if (rows == 4) {
     if (p.dv <= 64) launch_bias_attn<T, 32, 1, 2, TOut, MAPS>(p, grid, stream);
-    else if (MAPS == 2 && p.dv <= 128) launch_bias_attn<T, 32, 1, 4, TOut, MAPS>(p, grid, stream);
+    else if (p.dv <= 128) launch_bias_attn<T, 32, 1, 4, TOut, MAPS>(p, grid, stream);
     else launch_bias_attn<T, 32, 1, 8, TOut, MAPS>(p, grid, stream);
   } else if (rows == 8) {
-    if (p.dv <= 64) launch_bias_attn<T, 16, 1, 4, TOut, MAPS>(p, grid, stream);
-    else if (MAPS == 2 && p.dv <= 128) launch_bias_attn<T, 16, 1, 8, TOut, MAPS>(p, grid, stream);
-    else launch_bias_attn<T, 16, 1, 16, TOut, MAPS>(p, grid, stream);
+    if (p.dv <= 64) launch_bias_attn<T, 32, 2, 2, TOut, MAPS>(p, grid, stream);
+    else if (p.dv <= 128) launch_bias_attn<T, 32, 2, 4, TOut, MAPS>(p, grid, stream);
+    else launch_bias_attn<T, 32, 2, 8, TOut, MAPS>(p, grid, stream);
   } else {
     if (p.dv <= 32) launch_bias_attn<T, 8, 2, 4, TOut, MAPS>(p, grid, stream);
     else if (p.dv <= 64) launch_bias_attn<T, 8, 2, 8, TOut, MAPS>(p, grid, stream);
@@ -603,8 +620,9 @@ RL_EXPORT int rl_bias_attention(int cache_dtype, int out_dtype, const float* q, 
   if (n_splits > 1) {
     const dim3 mg(p.n_decode, (n_heads + 3) / 4);
     if (maps == 2) {
-      if (out_dtype == RL_F32) rl::launch_pdl(rl::bias_attn_merge_maps_kernel<float>, mg, 128, 0, stream, p);
-      else rl::launch_pdl(rl::bias_attn_merge_maps_kernel<__nv_bfloat16>, mg, 128, 0, stream, p);
+      const dim3 mg2(p.n_decode, n_heads);
+      if (out_dtype == RL_F32) rl::launch_pdl(rl::bias_attn_merge_maps_kernel<float>, mg2, 128, 0, stream, p);
+      else rl::launch_pdl(rl::bias_attn_merge_maps_kernel<__nv_bfloat16>, mg2, 128, 0, stream, p);
     } else if (out_dtype == RL_F32) rl::launch_pdl(rl::bias_attn_merge_kernel<float>, mg, 128, 0, stream, p);
     else rl::launch_pdl(rl::bias_attn_merge_kernel<__nv_bfloat16>, mg, 128, 0, stream, p);
   }
