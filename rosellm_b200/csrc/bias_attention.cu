@@ -507,7 +507,11 @@ static void launch_bias_attn(const BiasAttnParams& p, dim3 grid, cudaStream_t st
       raised = true;
     }
   }
-  launch_pdl(kernel, grid, BA_THREADS, smem, stream, p);
+  // What hides a tile's chain of dependent steps is other blocks on the SM: a grid that the common split (half of an SM's
+  // memory) does not hold at once, of blocks of which fewer than five fit there, takes all of it.
+  const long fit = (long)(114 * 1024 / (smem + 1024));
+  if (fit < 5 && (long)grid.x * grid.y * grid.z > 148 * fit) launch_pdl_all_shared(kernel, grid, BA_THREADS, smem, stream, p);
+  else launch_pdl(kernel, grid, BA_THREADS, smem, stream, p);
 }
 
 // rows: 32 (prompt tiles, and decoded tokens of large groups), 8 or 4 (decoded tokens)

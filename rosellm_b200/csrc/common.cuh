@@ -145,6 +145,26 @@ inline cudaError_t launch_pdl(void (*kernel)(KArgs...), dim3 grid, dim3 block, s
   return launch_pdl_split(true, kernel, grid, block, smem, stream, args...);
 }
 
+// One launch of a kernel that otherwise runs with the common split, with all of an SM's memory as shared memory: for
+// grids whose blocks would not all run at once otherwise.
+template <typename... KArgs, typename... Args>
+inline cudaError_t launch_pdl_all_shared(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t stream,
+                                         Args... args) {
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = grid;
+  cfg.blockDim = block;
+  cfg.dynamicSmemBytes = smem;
+  cfg.stream = stream;
+  cudaLaunchAttribute attr[2];
+  attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attr[0].val.programmaticStreamSerializationAllowed = 1;
+  attr[1].id = cudaLaunchAttributePreferredSharedMemoryCarveout;
+  attr[1].val.sharedMemCarveout = cudaSharedmemCarveoutMaxShared;
+  cfg.attrs = attr;
+  cfg.numAttrs = 2;
+  return note_launch(cudaLaunchKernelEx(&cfg, kernel, KArgs(args)...));
+}
+
 // Thread-block clusters: rank of this block, the barrier of all threads of the cluster, and
 // the address of a shared-memory location in another block of the cluster.
 __device__ __forceinline__ uint32_t cluster_rank() {
