@@ -208,7 +208,7 @@ class MixtureOfExperts(Part):
         z = full[:, :E]
         choice = dict(top=top, group_count=self.group_count, group_keep=self.group_keep, score=self.score, ids=ids,
                       weights=weights)
-        if n <= K.MOE_ROUTE_MAX_TOKENS and n * top <= K.MOE_TABLE_ROUTE_MAX_PAIRS:
+        if n <= K.MOE_ROUTE_FUSED_UP_TO and n * top <= K.MOE_TABLE_ROUTE_MAX_PAIRS:
             K.moe_select_route(z, self.correction, offsets=offsets, tiles=tiles, meta=meta, row_token=row_token,
                                place_of=place_of, place_weight=by_place, **choice)
         else:
