@@ -17,6 +17,7 @@ from .porovik import PorovikConfig
 from .fikevik import FikevikConfig
 from .soporax import SoporaxConfig
 from .vebotar import VebotarConfig
+from .kugadra import KugadraConfig
 
 __all__ = [
     "Architecture",
@@ -28,6 +29,7 @@ __all__ = [
     "FikevikConfig",
     "SoporaxConfig",
     "VebotarConfig",
+    "KugadraConfig",
     "ModelConfig",
     "load_config",
     "parse_config",

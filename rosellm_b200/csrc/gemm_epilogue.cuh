@@ -24,6 +24,9 @@ __device__ __forceinline__ float apply_act(float u, int act) {
   return u;
 }
 
+// Logits bounded smoothly by +-cap (cap <= 0: as they are).
+__device__ __forceinline__ float soft_capped(float v, float cap) { return cap > 0.f ? cap * tanhf(v / cap) : v; }
+
 template <typename TOut>
 __device__ __forceinline__ void store_out(TOut* out, size_t idx, float v, int residual) {
   out[idx] = from_f32<TOut>(v);
@@ -71,6 +74,7 @@ struct SampleArgs {
   int* host_ring;
   int ring_stride;
   unsigned int* ring_step;
+  float soft_cap;  // > 0: the logits are soft_cap * tanh(logit / soft_cap) before anything else
 };
 constexpr unsigned int SAMPLE_RING = 4;
 

@@ -352,7 +352,8 @@ __global__ __launch_bounds__(32 * KSPLIT * GROUPS) void gemm_rows_mma_kernel(
           const int m = t * 16 + hlf * 8 + g;
           const int mc = m < M ? m : 0;  // every lane takes part in the exchanges below
           const float temp = temp_of[t][hlf];
-          float s0 = apply_act(c[t][2 * hlf] + bias0, act), s1 = apply_act(c[t][2 * hlf + 1] + bias1, act);
+          float s0 = soft_capped(apply_act(c[t][2 * hlf] + bias0, act), sample.soft_cap);
+          float s1 = soft_capped(apply_act(c[t][2 * hlf + 1] + bias1, act), sample.soft_cap);
           if (temp > 0.f) {
             const uint64_t seed = (uint64_t)sample.seeds[mc];
             const uint32_t counter = (uint32_t)sample.counters[mc];
@@ -582,13 +583,14 @@ RL_EXPORT int rl_gemm_rows_bf16(int out_dtype, const void* A, long lda, const vo
 // written: out_ids[m] is what rl_sample would choose from row m of A W^T (+ bias) with the same
 // temperature, seed and counter (rows with top-k or top-p are not for this entry point).
 // best [M] and ticket [1] are scratch that is zero before the call and zero again after it.
-// host_ring != nullptr: the ids are also written to that pinned host memory (see SampleArgs).
+// host_ring != nullptr: the ids are also written to that pinned host memory (see SampleArgs).  soft_cap > 0: the logits
+// are soft_cap * tanh(logit / soft_cap).
 RL_EXPORT int rl_gemm_rows_bf16_sample(const void* A, long lda, const void* W, const float* bias, int M, int N, int K,
                                        const float* norm_x, long norm_ldx, const float* norm_gamma,
                                        const float* norm_beta, float norm_eps, const float* temperature,
                                        const long long* seeds, const int* counters, int* out_ids,
                                        unsigned long long* best, int* ticket, int* host_ring, int ring_stride,
-                                       unsigned int* ring_step, int* status, cudaStream_t stream) {
+                                       unsigned int* ring_step, float soft_cap, int* status, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if (M > 64) return -5;
   if (out_ids == nullptr || best == nullptr || ticket == nullptr) return -7;
@@ -601,7 +603,7 @@ RL_EXPORT int rl_gemm_rows_bf16_sample(const void* A, long lda, const void* W, c
   const rl::NormArgs norm{norm_x, norm_ldx, norm_gamma, norm_beta, norm_eps};
   const rl::KvScatter kv{};
   if (host_ring != nullptr && (ring_step == nullptr || ring_stride < M)) return -7;
-  const rl::SampleArgs sample{out_ids, temperature, seeds, counters, best, ticket, host_ring, ring_stride, ring_step};
+  const rl::SampleArgs sample{out_ids, temperature, seeds, counters, best, ticket, host_ring, ring_stride, ring_step, soft_cap};
   const __nv_bfloat16* a = (const __nv_bfloat16*)A;
   const __nv_bfloat16* w = (const __nv_bfloat16*)W;
   if (status != nullptr) {

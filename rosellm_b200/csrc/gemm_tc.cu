@@ -69,6 +69,8 @@ __device__ __noinline__ float sample_key_call(float logit, float inv_t, uint64_t
   return sample_key(logit, inv_t, seed, counter, index);
 }
 
+__device__ __noinline__ float soft_capped_call(float v, float cap) { return soft_capped(v, cap); }
+
 // What a launch is told beyond the tensor maps.
 struct PArgs {
   const float* bias;
@@ -334,20 +336,23 @@ __global__ __launch_bounds__(PTHREADS, 1) void gemm_tc_persistent_kernel(const _
           asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
           const float bias_c = c == part ? bias0 : bias1;
           const int col0 = n0 + c * 32;
-          if (!any_sampled) {
+          if (!any_sampled && sm.soft_cap <= 0.f) {
 #pragma unroll
             for (int i = 0; i < 32; ++i) {
               const float v = act_fn(__uint_as_float(r[i]) + __shfl_sync(0xffffffffu, bias_c, i), p.act);
               if (col0 + i < N) best = better(best, ArgMax{v, col0 + i});
             }
           } else {
-            // the noise is a call, not thirty-two inlined copies: the loop of the rows that take
+            // noise and bound are calls, not thirty-two inlined copies: the loop of the rows that take
             // the arg-max (above) stays short, and so does what the instruction cache must hold
 #pragma unroll
             for (int i = 0; i < 32; ++i) {
               float v = act_fn(__uint_as_float(r[i]) + __shfl_sync(0xffffffffu, bias_c, i), p.act);
-              const float key = sample_key_call(v, inv_t, seed, counter, (uint32_t)(col0 + i));
-              if (temp > 0.f) v = key;
+              if (sm.soft_cap > 0.f) v = soft_capped_call(v, sm.soft_cap);
+              if (any_sampled) {
+                const float key = sample_key_call(v, inv_t, seed, counter, (uint32_t)(col0 + i));
+                if (temp > 0.f) v = key;
+              }
               if (col0 + i < N) best = better(best, ArgMax{v, col0 + i});
             }
           }
@@ -874,7 +879,7 @@ RL_EXPORT int rl_gemm_tc(int out_dtype, const void* A, long lda, const void* W, 
 RL_EXPORT int rl_gemm_tc_sample(const void* A, long lda, const void* W, const float* bias, int M, int N, int K,
                                 const float* temperature, const long long* seeds, const int* counters, int* out_ids,
                                 unsigned long long* best, int* ticket, int* host_ring, int ring_stride,
-                                unsigned int* ring_step, int* status, cudaStream_t stream) {
+                                unsigned int* ring_step, float soft_cap, int* status, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if (K % 8 != 0 || lda % 8 != 0 || ((uintptr_t)A % 16) != 0 || ((uintptr_t)W % 16) != 0) return -2;
   if (out_ids == nullptr || best == nullptr || ticket == nullptr || status == nullptr) return -7;
@@ -882,7 +887,7 @@ RL_EXPORT int rl_gemm_tc_sample(const void* A, long lda, const void* W, const fl
   using namespace rl::tc;
   const rl::KvScatter kv{};
   if (host_ring != nullptr && (ring_step == nullptr || ring_stride < M)) return -7;
-  const rl::SampleArgs sample{out_ids, temperature, seeds, counters, best, ticket, host_ring, ring_stride, ring_step};
+  const rl::SampleArgs sample{out_ids, temperature, seeds, counters, best, ticket, host_ring, ring_stride, ring_step, soft_cap};
   const Cut cut = plan_cut(M, N, K, false, 0, 0, 0);
   return launch_persistent<float, EPI_SAMPLE, false>(A, lda, W, bias, nullptr, 0, M, N, K, RL_ACT_NONE, 0, kv, status, cut,
                                                      stream, sample);

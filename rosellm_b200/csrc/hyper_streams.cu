@@ -41,7 +41,7 @@ struct HyperStepParams {
   int top;
   const float* shared;   // [tokens, width] (row stride ld_shared) or null
   long ld_shared;
-  const float* sg;       // logits, one a token, stride ldsg
+  const float* sg;       // logits, one a token, stride ldsg; null: a factor of 1
   long ldsg;
 };
 
@@ -89,8 +89,8 @@ __global__ __launch_bounds__(256) void hyper_step_kernel(const HyperStepParams p
   }
   __syncthreads();
   const float* xr = p.x + (size_t)t * p.ldx;
-  float gate = 0.f;
-  if (WRITE && p.eo != nullptr && p.shared != nullptr) gate = 1.0f / (1.0f + expf(-p.sg[(size_t)t * p.ldsg]));
+  float gate = 1.f;
+  if (WRITE && p.eo != nullptr && p.shared != nullptr && p.sg != nullptr) gate = 1.0f / (1.0f + expf(-p.sg[(size_t)t * p.ldsg]));
   float ss = 0.f;
   for (int d = threadIdx.x * V; d < p.width; d += blockDim.x * V) {
     HyperVec<V> x[S], r[S], y;
@@ -205,7 +205,7 @@ RL_EXPORT int rl_hyper_step(int h_dtype, const float* x, long ldx, long x_copy, 
   const bool write = mix != nullptr, read = gamma != nullptr;
   if (copies < 1 || copies > 16 || width <= 0 || (!write && !read) || (write && out_w == nullptr) ||
       (write && y == nullptr && (eo == nullptr || place_of == nullptr || top <= 0)) || (read && (in_w == nullptr || h == nullptr)) ||
-      (!read && sum == nullptr) || (shared != nullptr && sg == nullptr))
+      (!read && sum == nullptr) || (shared == nullptr && sg != nullptr))
     return -2;
   if (read && width > 12000) return -3;
   const rl::HyperStepParams p{x, ldx, x_copy, x_new, ldn, y, ldy, mix, out_w, in_w, gamma, eps, h, ldh, sum, lds, n_tokens,

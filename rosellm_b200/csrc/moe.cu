@@ -2,7 +2,8 @@
 //
 // Routing (`moe_select_kernel`, one warp per token, float32): scores s = softmax(z) over all
 // experts, or (score_kind 1) s = sigmoid(z) of each expert by itself, or (score_kind 2) s = z; the choice is made on
-// s + correction, the weights are the chosen experts' s, with score_kind 2 the softmax over the chosen s alone.  With
+// s + correction, the weights are the chosen experts' s, with score_kind 2 the softmax over the chosen s alone;
+// with weight_scale > 0 the weights are divided by their sum (+ 1e-20) and multiplied by it.  With
 // groups, the experts form `group_count` equal groups of neighbours, a group's score is the
 // largest choice score in it, and only experts of the best `group_keep` groups can be chosen
 // (the others count as minus infinity).  Ties go to the lower index.
@@ -97,9 +98,9 @@ __device__ __forceinline__ void moe_layout_block(int n_pairs, int top, int n_exp
 // counted for each.  s_w, c_w, g_w: the warp's scratch in shared memory, E floats each (scores, choice scores, group
 // scores).
 __device__ __forceinline__ void moe_select_token(const float* __restrict__ zr, const float* __restrict__ correction, int E,
-                                                 int top, int group_count, int group_keep, int score_kind, float* s_w,
-                                                 float* c_w, float* g_w, int* ids_t, float* weights_t, int* counts,
-                                                 int lane) {
+                                                 int top, int group_count, int group_keep, int score_kind, float weight_scale,
+                                                 float* s_w, float* c_w, float* g_w, int* ids_t, float* weights_t,
+                                                 int* counts, int lane) {
   float sum = 1.f;
   if (score_kind == MOE_SCORE_SIGMOID) {
     for (int e = lane; e < E; e += 32) s_w[e] = 1.0f / (1.0f + expf(-zr[e]));
@@ -177,7 +178,14 @@ __device__ __forceinline__ void moe_select_token(const float* __restrict__ zr, c
     float total = 0.f;
     for (int j = lane; j < top; j += 32) total += expf(g_w[j] - mx);
     total = warp_sum(total);
-    for (int j = lane; j < top; j += 32) weights_t[j] = expf(g_w[j] - mx) / total;
+    for (int j = lane; j < top; j += 32) g_w[j] = weights_t[j] = expf(g_w[j] - mx) / total;
+    __syncwarp();
+  }
+  if (weight_scale > 0.f) {  // the chosen weights as shares of their sum, times a factor
+    float total = 0.f;
+    for (int j = lane; j < top; j += 32) total += g_w[j];
+    total = warp_sum(total) + 1e-20f;
+    for (int j = lane; j < top; j += 32) weights_t[j] = g_w[j] / total * weight_scale;
     __syncwarp();
   }
 }
@@ -185,15 +193,15 @@ __device__ __forceinline__ void moe_select_token(const float* __restrict__ zr, c
 __global__ __launch_bounds__(128) void moe_select_kernel(const float* __restrict__ z, long ldz,
                                                          const float* __restrict__ correction, int n_tokens,
                                                          int n_experts, int top, int group_count, int group_keep,
-                                                         int score_kind, int* __restrict__ ids, float* __restrict__ weights,
-                                                         int* __restrict__ counts) {
+                                                         int score_kind, float weight_scale, int* __restrict__ ids,
+                                                         float* __restrict__ weights, int* __restrict__ counts) {
   extern __shared__ float smem[];
   pdl_begin();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int t = blockIdx.x * 4 + warp;
   if (t >= n_tokens) return;
   float* s_w = smem + (size_t)warp * 3 * n_experts;
-  moe_select_token(z + (size_t)t * ldz, correction, n_experts, top, group_count, group_keep, score_kind, s_w,
+  moe_select_token(z + (size_t)t * ldz, correction, n_experts, top, group_count, group_keep, score_kind, weight_scale, s_w,
                    s_w + n_experts, s_w + 2 * n_experts, ids + (size_t)t * top, weights + (size_t)t * top, counts, lane);
 }
 
@@ -205,7 +213,8 @@ constexpr int MOE_ROUTE_MAX_TOKENS = 128;
 __global__ __launch_bounds__(1024, 1) void moe_select_route_kernel(const float* __restrict__ z, long ldz,
                                                                 const float* __restrict__ correction, int n_tokens,
                                                                 int n_experts, int top, int group_count, int group_keep,
-                                                                int score_kind, int* __restrict__ ids,
+                                                                int score_kind, float weight_scale,
+                                                                int* __restrict__ ids,
                                                                 float* __restrict__ weights, int* __restrict__ offsets,
                                                                 int* __restrict__ tiles, int* __restrict__ meta,
                                                                 int* __restrict__ row_token, int* __restrict__ place_of,
@@ -218,7 +227,7 @@ __global__ __launch_bounds__(1024, 1) void moe_select_route_kernel(const float* 
   __syncthreads();
   float* s_w = smem + (size_t)warp * 3 * n_experts;
   for (int t = warp; t < n_tokens; t += n_warps) {
-    moe_select_token(z + (size_t)t * ldz, correction, n_experts, top, group_count, group_keep, score_kind, s_w,
+    moe_select_token(z + (size_t)t * ldz, correction, n_experts, top, group_count, group_keep, score_kind, weight_scale, s_w,
                      s_w + n_experts, s_w + 2 * n_experts, ids + (size_t)t * top, weights + (size_t)t * top, count_s, lane);
     __syncwarp();
   }
@@ -560,7 +569,7 @@ __global__ __launch_bounds__(256) void moe_rows_kernel(const __nv_bfloat16* __re
 }
 
 // y[t] (+)= sum_j weights[t, j] * eo[place_of[t, j]], j in order (weights null: plain sum), + sigmoid(sg[t]) *
-// shared[t] where given (shared: float32 [tokens, hidden]; sg: one logit a token, stride ldsg).
+// shared[t] where given (shared: float32 [tokens, hidden]; sg: one logit a token, stride ldsg; null: a factor of 1).
 __global__ __launch_bounds__(256) void moe_combine_kernel(const float* __restrict__ eo,
                                                           const float* __restrict__ weights,
                                                           const int* __restrict__ place_of, float* __restrict__ y,
@@ -570,7 +579,7 @@ __global__ __launch_bounds__(256) void moe_combine_kernel(const float* __restric
   pdl_begin();
   const int t = blockIdx.x;
   if (t >= n_tokens) return;
-  const float gate = shared != nullptr ? 1.0f / (1.0f + expf(-sg[(size_t)t * ldsg])) : 0.f;
+  const float gate = sg != nullptr ? 1.0f / (1.0f + expf(-sg[(size_t)t * ldsg])) : 1.0f;
   for (int d = threadIdx.x; d < hidden; d += blockDim.x) {
     float acc = 0.f;
     for (int j = 0; j < top; ++j)
@@ -587,8 +596,8 @@ __global__ __launch_bounds__(256) void moe_combine_kernel(const float* __restric
 // z: float32 router logits [tokens, experts] (row stride ldz).  ids, weights: [tokens * top].
 // counts: [experts], zero on entry; holds the experts' pair counts afterwards.
 RL_EXPORT int rl_moe_select(const float* z, long ldz, const float* correction, int n_tokens, int n_experts, int top,
-                            int group_count, int group_keep, int score_kind, int* ids, float* weights, int* counts,
-                            cudaStream_t stream) {
+                            int group_count, int group_keep, int score_kind, float weight_scale, int* ids, float* weights,
+                            int* counts, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
   if (n_experts <= 0 || n_experts > 2048 || top <= 0 || top > n_experts || score_kind < 0 || score_kind > 2) return -2;
   if (group_count < 1 || n_experts % group_count != 0 || group_keep < 1 || group_keep > group_count ||
@@ -598,7 +607,7 @@ RL_EXPORT int rl_moe_select(const float* z, long ldz, const float* correction, i
   if (smem > 48 * 1024)
     cudaFuncSetAttribute(rl::moe_select_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   rl::launch_pdl(rl::moe_select_kernel, (n_tokens + 3) / 4, 128, smem, stream, z, ldz, correction, n_tokens, n_experts,
-                 top, group_count, group_keep, score_kind, ids, weights, counts);
+                 top, group_count, group_keep, score_kind, weight_scale, ids, weights, counts);
   RL_CHECK_LAUNCH();
   return 0;
 }
@@ -606,7 +615,8 @@ RL_EXPORT int rl_moe_select(const float* z, long ldz, const float* correction, i
 // Routing and layout in one launch: what rl_moe_select and rl_moe_plan leave, for at most 128 tokens (-3 beyond).  No
 // counters in global memory are used.  place_weight: null, or float32 [tokens * top] that receives the weights by place.
 RL_EXPORT int rl_moe_select_route(const float* z, long ldz, const float* correction, int n_tokens, int n_experts, int top,
-                                  int group_count, int group_keep, int score_kind, int* ids, float* weights, int* offsets,
+                                  int group_count, int group_keep, int score_kind, float weight_scale, int* ids,
+                                  float* weights, int* offsets,
                                   int* tiles, int* meta, int* row_token, int* place_of, float* place_weight,
                                   cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
@@ -621,7 +631,7 @@ RL_EXPORT int rl_moe_select_route(const float* z, long ldz, const float* correct
   if (warps > n_tokens) warps = n_tokens;
   if (warps < 1) return -3;
   rl::launch_pdl(rl::moe_select_route_kernel, 1, warps * 32, (size_t)warps * 3 * n_experts * sizeof(float), stream, z, ldz,
-                 correction, n_tokens, n_experts, top, group_count, group_keep, score_kind, ids, weights, offsets, tiles,
+                 correction, n_tokens, n_experts, top, group_count, group_keep, score_kind, weight_scale, ids, weights, offsets, tiles,
                  meta, row_token, place_of, place_weight);
   RL_CHECK_LAUNCH();
   return 0;
@@ -685,14 +695,14 @@ RL_EXPORT int rl_moe_max_tiles(int n_pairs, int n_experts) {
 // w_down: [experts][hidden][ff]; act: scratch [pairs, ff] (row stride lda); eo: float32 scratch
 // [pairs, hidden]; y: float32 [tokens, hidden] (row stride ldy), overwritten or (add) added to.
 // place_weight (by place) scales the experts' inputs, weights (by pair) their outputs; either may be null.
-// shared (or null): float32 [tokens, hidden], added times sigmoid(sg[token]).
+// shared (or null): float32 [tokens, hidden], added, times sigmoid(sg[token]) where sg is given.
 RL_EXPORT int rl_moe_experts(int dtype, const void* h, long ldh, const void* w_gu, const void* w_down, const int* tiles,
                              const int* meta, const int* row_token, const int* place_of, const float* weights,
                              const float* place_weight, void* act, long lda, float* eo, float* y, long ldy, int n_tokens,
                              int hidden, int ff, int n_experts, int top, int kind, float alpha, float limit, int add,
                              const float* shared, long lds, const float* sg, long ldsg, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
-  if (hidden <= 0 || ff <= 0 || kind < 0 || kind > RL_UNIT_LAST || (shared != nullptr && sg == nullptr)) return -2;
+  if (hidden <= 0 || ff <= 0 || kind < 0 || kind > RL_UNIT_LAST || (shared == nullptr && sg != nullptr)) return -2;
   const bool pair = kind < RL_UNIT_FIRST;
   const int max_tiles = rl_moe_max_tiles(n_tokens * top, n_experts);
   const dim3 g1(max_tiles, (ff + rl::TG_N - 1) / rl::TG_N), g2(max_tiles, (hidden + rl::TG_N - 1) / rl::TG_N);

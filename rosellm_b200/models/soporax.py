@@ -38,7 +38,7 @@ def _mixer_spec(kind: str, mx, m: str, width: int, eps: float) -> PartSpec:
             "latent_attention",
             dict(hidden_size=width, num_heads=mx.heads, plain_dim=mx.dim, rot_dim=mx.rot_dim, value_dim=mx.vdim,
                  kv_rank=mx.kv_rank, scale=mx.scale, rot_dims=0 if rot is None else rot.dims,
-                 rot_base=10000.0 if rot is None else rot.base, norm_eps=eps, sink=False, q_rank=mx.q_rank, gate=True,
+                 rot_base=10000.0 if rot is None else rot.base, norm_eps=eps, sink=False, q_rank=mx.q_rank, gate="element",
                  rot_scaling=None if rot is None else rot.scaling_params()),
             tensors)
     common = dict(hidden_size=width, num_heads=mx.heads, num_kv_heads=mx.kv_heads, key_dim=mx.dim, value_dim=mx.vdim,

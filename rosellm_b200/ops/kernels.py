@@ -130,13 +130,13 @@ def _lib() -> ctypes.CDLL:
                                      I, I, I, I, I, I, P, P]
         lib.rl_gemm_rows_bf16.argtypes = [I, P, L, P, P, P, L, I, I, I, I, I, P, L, P, P, F, P, P, I, P, P, P,
                                           I, I, I, I, I, I, P, P]
-        lib.rl_gemm_rows_bf16_sample.argtypes = [P, L, P, P, I, I, I, P, L, P, P, F, P, P, P, P, P, P, P, I, P, P, P]
+        lib.rl_gemm_rows_bf16_sample.argtypes = [P, L, P, P, I, I, I, P, L, P, P, F, P, P, P, P, P, P, P, I, P, F, P, P]
         lib.rl_host_memory_on_device.argtypes = [P]
         lib.rl_host_memory_on_device.restype = ctypes.c_ulonglong
         lib.rl_gemm_rows_bulk_enable.argtypes = [I]
         lib.rl_gemm_rows_bulk_enable.restype = None
         lib.rl_gemm_tc.argtypes = [I, P, L, P, P, P, L, I, I, I, I, I, P, P, I, P, P, P, I, I, I, I, I, I, P, P]
-        lib.rl_gemm_tc_sample.argtypes = [P, L, P, P, I, I, I, P, P, P, P, P, P, P, I, P, P, P]
+        lib.rl_gemm_tc_sample.argtypes = [P, L, P, P, I, I, I, P, P, P, P, P, P, P, I, P, F, P, P]
         lib.rl_gemm_tc_cut.argtypes = [I, P, L, P, P, P, L, I, I, I, I, I, P, P, I, P, P, P, I, I, I, I, I, I, P, I, I, P]
         lib.rl_gemm_tc_rows.argtypes = [I, P, L, P, P, P, L, I, I, I, I, I, P, P, I, P, P, P, I, I, I, I, I, I, P, P]
         lib.rl_gemm_tc_rows_fits.argtypes = [I, I, I]
@@ -160,20 +160,23 @@ def _lib() -> ctypes.CDLL:
         lib.rl_latent_kv_write.argtypes = [I, P, L, P, F, P, I, P, P, I, P, P, P, I, I, I, I, I, I, F, P, P]
         lib.rl_latent_q_rope.argtypes = [I, P, L, I, I, P, L, I, I, I, I, P, P, I, I, F, P]
         lib.rl_latent_attention.argtypes = [I, P, L, P, P, I, P, P, P, P, L, P, I, I, I, I, F, P, I, P, I, I, I, P, P, I, P, P]
-        lib.rl_head_linear.argtypes = [I, P, L, L, P, L, L, L, P, L, L, I, I, I, I, P, L, L, P]
+        lib.rl_head_linear.argtypes = [I, P, L, L, P, L, L, L, P, L, L, I, I, I, I, P, L, L, L, P]
         lib.rl_gated_act.argtypes = [I, P, L, I, P, L, I, I, I, F, F, P]
         lib.rl_token_gate.argtypes = [I, P, L, P, P, L, I, I, P, L, I, I, I, P, I, P, P]
-        lib.rl_moe_select.argtypes = [P, L, P, I, I, I, I, I, I, P, P, P, P]
+        lib.rl_moe_select.argtypes = [P, L, P, I, I, I, I, I, I, F, P, P, P, P]
         lib.rl_moe_plan.argtypes = [P, P, P, P, P, P, P, P, P, P, I, I, I, P]
         lib.rl_moe_max_tiles.argtypes = [I, I]
         lib.rl_moe_experts.argtypes = [I, P, L, P, P, P, P, P, P, P, P, P, L, P, P, L, I, I, I, I, I, I, F, F, I, P, L, P, L, P]
-        lib.rl_moe_select_route.argtypes = [P, L, P, I, I, I, I, I, I, P, P, P, P, P, P, P, P, P]
+        lib.rl_moe_select_route.argtypes = [P, L, P, I, I, I, I, I, I, F, P, P, P, P, P, P, P, P, P]
         lib.rl_hyper_step.argtypes = [I, P, L, L, P, L, P, L, P, P, P, P, F, P, L, P, L, I, I, I, P, P, P, I, P, L, P, L, P]
         lib.rl_embed_pair.argtypes = [I, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, P, P, P, I, P]
         lib.rl_rmsnorm_add_norm.argtypes = [I, P, L, P, P, L, P, P, L, I, I, F, F, P]
         lib.rl_recurrence.argtypes = [I, I, P, L, I, I, I, I, I, I, P, P, P, I, P, P, P, L, P, P, P, P, I, I, I, I, I, F, F, F,
                                       L, I, F, F, F, F, P, P]
         lib.rl_recurrence_record.argtypes = [I, I, I, P, P, P]
+        lib.rl_lightning.argtypes = [P, L, I, I, I, I, P, P, L, P, P, P, I, P, I, P, P, I, I, I, I, P]
+        lib.rl_rmsnorm_gate.argtypes = [I, P, L, P, L, P, P, L, I, I, F, P]
+        lib.rl_soft_cap.argtypes = [P, L, F, P]
         lib.rl_bias_attention_shape.argtypes = [I, I, P, P]
         lib.rl_bias_attention.argtypes = [I, I, P, L, P, L, P, P, L, P, P, P, P, I, I, P, I, P, L, I, I, I, I, I, I, I, I,
                                           F, F, I, P, P, I, P, P, I, I, P, P, I, I, I, P, F, F, P]
@@ -192,7 +195,7 @@ def _lib() -> ctypes.CDLL:
                      "rl_rmsnorm_add_norm", "rl_recurrence", "rl_recurrence_record", "rl_bias_attention_shape", "rl_bias_attention",
                      "rl_bias_kv_store", "rl_qkv_norm_rotate", "rl_gated_join_norm", "rl_stream_inject", "rl_gate_mul",
                      "rl_moe_table_select", "rl_stream_inject_norm", "rl_moe_table_route",
-                     "rl_moe_select_route", "rl_hyper_step"):
+                     "rl_moe_select_route", "rl_hyper_step", "rl_lightning", "rl_rmsnorm_gate", "rl_soft_cap"):
             getattr(lib, name).restype = I
         for name in ("rl_copy_to_device", "rl_event_record", "rl_embed", "rl_layernorm", "rl_gemm_simt", "rl_gemm_tc", "rl_gemm_tc_sample", "rl_gemm_tc_cut", "rl_gemm_tc_rows", "rl_gemm_tc_rows_fits",
                      "rl_gemm_rows_smem", "rl_gemm_rows_smem_fits",
@@ -595,12 +598,12 @@ def sampling_product_possible(rows: int, n_out: int, k: int, dtype: torch.dtype,
     return path == "mma" or (path == "tc" and not with_temperature)
 
 
-def linear_sample(a, weight, bias, into: SampleInto) -> None:
+def linear_sample(a, weight, bias, into: SampleInto, soft_cap: float = 0.0) -> None:
     """``into.out_ids[r]`` = the token ``sample`` would choose from row r of ``a @ weight.T + bias``
     (arg-max, or with a temperature the arg-max of logit / temperature + Gumbel noise), without
     the logits being written anywhere.  bfloat16, where ``sampling_product_possible``;
     ``a`` may be a ``NormInput`` as for ``linear``.  Rows with top-k or top-p need their logits:
-    they are not for this call."""
+    they are not for this call.  ``soft_cap`` > 0: a logit is soft_cap * tanh(logit / soft_cap)."""
     norm = a if isinstance(a, NormInput) else None
     _need(weight, "weight", torch.bfloat16)
     n, k = weight.shape
@@ -656,15 +659,23 @@ def linear_sample(a, weight, bias, into: SampleInto) -> None:
     if path == "tc":
         rc = _lib().rl_gemm_tc_sample(a_ptr, lda, _ptr(weight), _ptr(bias), m, n, k, _ptr(into.temperature),
                                       _ptr(into.seeds), _ptr(into.counters), _ptr(into.out_ids), _ptr(bufs[0]),
-                                      _ptr(bufs[1]), *ring, _ptr(status_word(weight.device)), _stream())
+                                      _ptr(bufs[1]), *ring, float(soft_cap), _ptr(status_word(weight.device)), _stream())
         if rc in (-10, -11):
             raise KernelError("linear_sample: the driver refused to encode a TMA tensor map for these operands")
         _ok(rc, "linear_sample (tcgen05)")
         return
     rc = _lib().rl_gemm_rows_bf16_sample(a_ptr, lda, _ptr(weight), _ptr(bias), m, n, k, *nx, _ptr(into.temperature),
                                          _ptr(into.seeds), _ptr(into.counters), _ptr(into.out_ids), _ptr(bufs[0]),
-                                         _ptr(bufs[1]), *ring, _ptr(status_word(weight.device)), _stream())
+                                         _ptr(bufs[1]), *ring, float(soft_cap), _ptr(status_word(weight.device)), _stream())
     _ok(rc, "linear_sample")
+
+
+def soft_cap(logits, cap: float) -> None:
+    """logits = cap * tanh(logits / cap), in place (float32, contiguous)."""
+    _need(logits, "logits", torch.float32)
+    if not cap > 0:
+        raise KernelError("soft_cap: the bound must be positive")
+    _ok(_lib().rl_soft_cap(_ptr(logits), logits.numel(), float(cap), _stream()), "soft_cap")
 
 
 def rows_bulk_kernel(on: bool) -> None:
@@ -1085,12 +1096,13 @@ def latent_attention(q, pool, block_table, q_start, kv_len, slots, out, *, sink,
 
 
 def head_linear(inp, w, out, *, n_tokens: int, n_heads: int, k: int, n: int, in_strides, w_strides, out_strides,
-                gate=None, gate_strides=(0, 0)) -> None:
+                gate=None, gate_strides=(0, 0, 1)) -> None:
     """out[t, h, :n] = inp[t, h, :k] @ W_h for every head: element (t, h, i) of ``inp`` at
     ``t*in_strides[0] + h*in_strides[1] + i``, element (h, i, j) of ``w`` at ``h*w_strides[0] +
     i*w_strides[1] + j*w_strides[2]``, element (t, h, j) of ``out`` at ``t*out_strides[0] +
     h*out_strides[1] + j`` (strides in elements; the tensors give base addresses and dtype).  ``gate``: float32
-    logits, element (t, h, j) at ``t*gate_strides[0] + h*gate_strides[1] + j``: the result times their sigmoid."""
+    logits, element (t, h, j) at ``t*gate_strides[0] + h*gate_strides[1] + j*gate_strides[2]`` (a last stride of 0: one
+    logit a head): the result times their sigmoid."""
     _need(inp, "inp", contiguous=False)
     _need(w, "w", inp.dtype)
     _need(out, "out", inp.dtype, contiguous=False)
@@ -1098,7 +1110,7 @@ def head_linear(inp, w, out, *, n_tokens: int, n_heads: int, k: int, n: int, in_
         _need(gate, "gate", torch.float32, contiguous=False)
     rc = _lib().rl_head_linear(_code(inp), _ptr(inp), in_strides[0], in_strides[1], _ptr(w), w_strides[0], w_strides[1],
                                w_strides[2], _ptr(out), out_strides[0], out_strides[1], n_tokens, n_heads, k, n,
-                               _ptr(gate), gate_strides[0], gate_strides[1], _stream())
+                               _ptr(gate), *gate_strides, _stream())
     _ok(rc, "head_linear")
 
 
@@ -1182,11 +1194,12 @@ MOE_SCORES = {"softmax": 0, "sigmoid": 1, "chosen_softmax": 2}
 
 
 def moe_select(z, correction, *, top: int, group_count: int, group_keep: int, ids, weights, counts,
-               score: int = 0) -> None:
+               score: int = 0, weight_scale: float = 0.0) -> None:
     """Routing of every row of the float32 router logits ``z`` [tokens, experts]: see csrc/moe.cu.
     ``ids`` int32 and ``weights`` float32 [tokens * top]; ``counts`` int32 [experts], zero on entry.
     ``score``: 0 softmax over the experts, 1 each expert's sigmoid, 2 the choice by the logits and the softmax over the
-    chosen experts' logits alone."""
+    chosen experts' logits alone.  ``weight_scale`` > 0: the weights are divided by their sum (+ 1e-20) and multiplied
+    by it."""
     _need(z, "z", torch.float32, contiguous=False)
     n, n_experts = z.shape
     for t, name, dt in ((ids, "ids", torch.int32), (weights, "weights", torch.float32), (counts, "counts", torch.int32)):
@@ -1194,7 +1207,7 @@ def moe_select(z, correction, *, top: int, group_count: int, group_keep: int, id
     if correction is not None:
         _need(correction, "correction", torch.float32)
     rc = _lib().rl_moe_select(_ptr(z), z.stride(0), _ptr(correction), n, n_experts, top, group_count, group_keep,
-                              int(score), _ptr(ids), _ptr(weights), _ptr(counts), _stream())
+                              int(score), float(weight_scale), _ptr(ids), _ptr(weights), _ptr(counts), _stream())
     if rc in (-2, -3):
         raise KernelError(f"moe_select: {n_experts} experts, top {top}, {group_keep} of {group_count} groups not taken")
     _ok(rc, "moe_select")
@@ -1207,7 +1220,7 @@ MOE_ROUTE_FUSED_UP_TO = 32
 
 
 def moe_select_route(z, correction, *, top: int, group_count: int, group_keep: int, score: int, ids, weights, offsets,
-                     tiles, meta, row_token, place_of, place_weight=None) -> None:
+                     tiles, meta, row_token, place_of, place_weight=None, weight_scale: float = 0.0) -> None:
     """``moe_select`` and ``moe_plan`` in one launch, for at most ``MOE_ROUTE_MAX_TOKENS`` tokens: the same ``ids``,
     ``weights``, ``offsets``, ``tiles``, ``meta``, ``row_token``, ``place_of`` and (given) ``place_weight``."""
     _need(z, "z", torch.float32, contiguous=False)
@@ -1224,7 +1237,7 @@ def moe_select_route(z, correction, *, top: int, group_count: int, group_keep: i
             or (place_weight is not None and place_weight.numel() < n * top):
         raise KernelError("moe_select_route: the outputs are too small")
     rc = _lib().rl_moe_select_route(_ptr(z), z.stride(0), _ptr(correction), n, n_experts, top, group_count, group_keep,
-                                    int(score), _ptr(ids), _ptr(weights), _ptr(offsets), _ptr(tiles), _ptr(meta),
+                                    int(score), float(weight_scale), _ptr(ids), _ptr(weights), _ptr(offsets), _ptr(tiles), _ptr(meta),
                                     _ptr(row_token), _ptr(place_of), _ptr(place_weight), _stream())
     if rc in (-2, -3):
         raise KernelError(f"moe_select_route: {n} tokens, {n_experts} experts, top {top}, {group_keep} of {group_count} "
@@ -1299,7 +1312,7 @@ def moe_experts(h, w_gate_up, w_down, tiles, meta, row_token, place_of, weights,
     ``y`` float32 [tokens, hidden] (``add``: added to it; ``None``: no sum, the experts' outputs stay in ``eo`` by place).
     ``gate``: a code of ``GATES`` (two input projections) or of ``UNITS`` (one: ``w_gate_up`` is then [experts * ff,
     hidden]).  ``shared`` float32 [tokens, hidden] and ``shared_gate`` float32 [tokens] (a column of a matrix will do):
-    added times the logit's sigmoid.  ``weights`` (by pair) weight the experts'
+    added times the logit's sigmoid (``shared_gate`` ``None``: as it is).  ``weights`` (by pair) weight the experts'
     outputs; ``place_weight`` (by place, from ``moe_plan``) their inputs instead; either may be ``None``.  ``w_gate_up`` [experts * 2 * ff, hidden]
     (per expert: gate rows, then up rows), ``w_down`` [experts * hidden, ff]."""
     _need(h, "h", contiguous=False)
@@ -1316,14 +1329,15 @@ def moe_experts(h, w_gate_up, w_down, tiles, meta, row_token, place_of, weights,
         raise KernelError("moe_experts: shapes do not fit")
     if shared is not None:
         _need(shared, "shared", torch.float32, contiguous=False)
-        _need(shared_gate, "shared_gate", torch.float32, contiguous=False)
-        if tuple(shared.shape) != (n, hidden) or shared.stride(1) != 1 or shared_gate.shape != (n,):
+        if shared_gate is not None:
+            _need(shared_gate, "shared_gate", torch.float32, contiguous=False)
+        if tuple(shared.shape) != (n, hidden) or shared.stride(1) != 1 or (shared_gate is not None and shared_gate.shape != (n,)):
             raise KernelError("moe_experts: the shared feed-forward's output or gate has another shape")
     rc = _lib().rl_moe_experts(_code(h), _ptr(h), h.stride(0), _ptr(w_gate_up), _ptr(w_down), _ptr(tiles), _ptr(meta),
                                _ptr(row_token), _ptr(place_of), _ptr(weights), _ptr(place_weight), _ptr(act), act.stride(0), _ptr(eo), _ptr(y),
                                0 if y is None else y.stride(0), n, hidden, ff, n_experts, top, gate, float(alpha), float(limit),
                                int(add), _ptr(shared), 0 if shared is None else shared.stride(0), _ptr(shared_gate),
-                               0 if shared is None else shared_gate.stride(0), _stream())
+                               0 if shared_gate is None else shared_gate.stride(0), _stream())
     _ok(rc, "moe_experts")
     global _launches
     _launches += 2 if y is not None else 1
@@ -1375,10 +1389,11 @@ def hyper_step(x, y, *, copies: int, write=None, x_new=None, read=None, gamma=No
         _need(y.place_of, "y.place_of", torch.int32)
         if y.eo.numel() < n * y.top * width or y.place_of.numel() < n * y.top:
             raise KernelError("hyper_step: the experts' outputs are too small")
-        if y.shared is not None and (tuple(y.shared.shape) != (n, width) or y.shared.stride(1) != 1 or y.shared_gate.shape != (n,)):
+        if y.shared is not None and (tuple(y.shared.shape) != (n, width) or y.shared.stride(1) != 1
+                                     or (y.shared_gate is not None and y.shared_gate.shape != (n,))):
             raise KernelError("hyper_step: the shared feed-forward's output or gate has another shape")
         ex = (_ptr(y.eo), _ptr(y.weights), _ptr(y.place_of), y.top, _ptr(y.shared), 0 if y.shared is None else y.shared.stride(0),
-              _ptr(y.shared_gate), 0 if y.shared is None else y.shared_gate.stride(0))
+              _ptr(y.shared_gate), 0 if y.shared_gate is None else y.shared_gate.stride(0))
     elif write is not None:
         _need(y, "y", torch.float32, contiguous=False)
         if tuple(y.shape) != (n, width) or y.stride(1) != 1:
@@ -1520,6 +1535,56 @@ def recurrence(mode: int, proj, offsets: dict, state, out, q_start, slots, prep,
     _ok(rc, "recurrence")
     global _launches
     _launches += 3 if mode == 3 else 2
+
+
+LIGHTNING_CHUNK = 64  # tokens a chunk (csrc/lightning.cu), a tile of the step's wide tiles
+
+
+def lightning(proj, offsets: dict, powers, state, q_start, slots, chunks, out, *, n_heads: int, dk: int, dv: int, tiles,
+              n_tiles: int, decode_reqs, n_decode: int, silu: bool = True, tensor_cores: bool = False) -> None:
+    """One step of linear attention with a fixed decay a head (csrc/lightning.cu) for every request of the step.
+    ``proj`` float32 [tokens, columns], ``offsets`` the first column of ``q``, ``k`` and ``v``; ``powers`` float32
+    [heads, 65]: the decays' powers 0 to 64; ``state`` float32 [slots, heads, dk, dv]; ``chunks`` float32 scratch of
+    n_tiles * heads * dk * dv floats (``None`` without portions); ``out`` float32 [tokens, heads * dv]; ``tiles``: the
+    step's 64-token tiles.  ``silu``: applied to the three projections.  ``tensor_cores``: portions of prompts with
+    queries, keys and values as bfloat16 operands."""
+    for t, name in ((powers, "powers"), (state, "state"), (out, "out")):
+        _need(t, name, torch.float32)
+    _need(proj, "proj", torch.float32, contiguous=False)
+    n = proj.shape[0]
+    if proj.stride(1) != 1 or tuple(powers.shape) != (n_heads, LIGHTNING_CHUNK + 1) or tuple(state.shape[1:]) != (n_heads, dk, dv) \
+            or tuple(out.shape) != (n, n_heads * dv):
+        raise KernelError("lightning: shapes do not fit")
+    off = [int(offsets[k]) for k in ("q", "k", "v")]
+    if any(o < 0 or o + w > proj.shape[1] for o, w in zip(off, (n_heads * dk, n_heads * dk, n_heads * dv))):
+        raise KernelError("lightning: a projection lies outside the matrix")
+    if n_tiles:
+        _need(chunks, "chunks", torch.float32)
+        if chunks.numel() < n_tiles * n_heads * dk * dv:
+            raise KernelError("lightning: scratch too small")
+    rc = _lib().rl_lightning(_ptr(proj), proj.stride(0), *off, int(silu), _ptr(powers), _ptr(state), state.stride(0),
+                             _ptr(q_start), _ptr(slots), _ptr(tiles), n_tiles, _ptr(decode_reqs), n_decode, _ptr(chunks),
+                             _ptr(out), n_heads, dk, dv, int(tensor_cores), _stream())
+    if rc == -2:
+        raise KernelError(f"lightning: sizes not taken (key size {dk}, value size {dv}: up to 256 each)")
+    _ok(rc, "lightning")
+    global _launches
+    _launches += (3 if n_tiles else 0) + (1 if n_decode else 0) - 1
+
+
+def rmsnorm_gate(x, gate, gamma, eps: float, out) -> None:
+    """out = x / sqrt(mean(x^2) + eps) * gamma * sigmoid(gate), row by row; ``x`` and ``gate`` float32 (views with a row
+    stride will do), ``out`` float32 or bfloat16."""
+    for t, name in ((x, "x"), (gate, "gate")):
+        _need(t, name, torch.float32, contiguous=False)
+    _need(gamma, "gamma", torch.float32)
+    _need(out, "out", contiguous=False)
+    n, width = x.shape
+    if tuple(gate.shape) != (n, width) or tuple(out.shape) != (n, width) or gamma.numel() != width \
+            or any(t.stride(1) != 1 for t in (x, gate, out)):
+        raise KernelError("rmsnorm_gate: shapes differ, or rows are not contiguous")
+    _ok(_lib().rl_rmsnorm_gate(_code(out), _ptr(x), x.stride(0), _ptr(gate), gate.stride(0), _ptr(gamma), _ptr(out), out.stride(0),
+                               n, width, float(eps), _stream()), "rmsnorm_gate")
 
 
 # ---- attention with a distance bias over rows of [key | value] -------------------------------------

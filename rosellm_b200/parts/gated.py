@@ -70,15 +70,18 @@ class MixtureOfExperts(Part):
     (``score="chosen_softmax"``) ``s = z``, where the weights are the softmax over the chosen scores alone; the choice is made on ``s + correction`` (where the
     model has one), restricted, with groups, to the experts of the ``group_keep`` groups (of
     ``group_count`` equal groups of neighbours) whose best choice score is largest; the chosen
-    experts' outputs are summed with their scores ``s`` as weights (not renormalised); with
+    experts' outputs are summed with their scores ``s`` as weights (not renormalised, unless ``weight_scale`` is given:
+    then the chosen scores are divided by their sum + 1e-20 and multiplied by it); with
     ``weight_input`` the weight multiplies the expert's input instead: the sum of ``expert(s * h)``.
     ``routing="table"``: no router; row ``token id`` of an integer table ``[vocab_size, top]`` (tensor ``table``; the
     entries of a row differ) names the token's experts, each with weight ``1 / top``.
     ``gate`` may also name an activation of one input projection (``relu_squared``): an expert is then ``W_down act(W_up
     h)`` and its tensor ``up_weight`` [experts * inner, hidden].
-    ``shared_inner`` > 0: a feed-forward of that inner size and of the same form (one input projection) runs for
-    every token and is added times ``sigmoid(W_sg h)``, one number a token (tensors ``shared_up_weight``,
-    ``shared_down_weight``, ``shared_gate_weight`` [1, hidden], the last in one product with the router).
+    ``shared_inner`` > 0: a feed-forward of that inner size and of the same form runs for every token and is added.
+    With experts of one input projection it is weighted by ``sigmoid(W_sg h)``, one number a token (tensors
+    ``shared_up_weight``, ``shared_down_weight``, ``shared_gate_weight`` [1, hidden], the last in one product with the
+    router); with gated experts it is added as it is (``shared_gate_up_weight`` [2 * inner, hidden],
+    ``shared_down_weight``).
     Routing, the experts' layout and their products all run on the device
     (csrc/moe.cu): a step's launches follow from its token count alone.
     Experts' tensors: ``gate_up_weight`` [experts * 2 * inner, hidden] (per expert the gate rows,
@@ -92,7 +95,8 @@ class MixtureOfExperts(Part):
     def __init__(self, hidden_size: int, inner_size: int, num_experts: int, top: int, group_count: int = 1,
                  group_keep: int = 1, gate: str = "silu", alpha: float = 1.0, limit: float = 0.0,
                  correction: bool = False, score: str = "softmax", weight_input: bool = False,
-                 routing: str = "router", vocab_size: int = 0, shared_inner: int = 0) -> None:
+                 routing: str = "router", vocab_size: int = 0, shared_inner: int = 0,
+                 weight_scale: float | None = None) -> None:
         if routing not in ("router", "table"):
             raise ValueError(f"mixture of experts: routing {routing!r}; 'router' or 'table'")
         if routing == "table" and (vocab_size <= 0 or correction or group_count != 1):
@@ -121,19 +125,26 @@ class MixtureOfExperts(Part):
         self.gated = gate not in K.UNITS
         self.gate, self.alpha, self.limit = (_gate(gate) if self.gated else K.UNITS[gate]), float(alpha), float(limit)
         self.shared_inner, self.shared_padded = int(shared_inner), -(-int(shared_inner) // 8) * 8
-        if shared_inner and (self.gated or routing != "router" or weight_input):
-            raise ValueError("mixture of experts: a shared feed-forward goes with experts of one input projection chosen by "
-                             "a router, whose outputs are weighted")
-        self.shared_act = K.ACTIVATIONS[gate] if shared_inner else None
+        if shared_inner and (routing != "router" or weight_input):
+            raise ValueError("mixture of experts: a shared feed-forward goes with experts chosen by a router, whose outputs "
+                             "are weighted")
+        if weight_scale is not None and (weight_scale <= 0 or routing != "router"):
+            raise ValueError("mixture of experts: a positive factor of the chosen weights, and a router")
+        self.weight_scale = 0.0 if weight_scale is None else float(weight_scale)
+        self.shared_act = K.ACTIVATIONS[gate] if shared_inner and not self.gated else None
+        self.gated_shared = bool(shared_inner) and self.gated
         self.has_correction = bool(correction)
         self.router_weight = self.correction = self.gate_up_weight = self.down_weight = self.table = None
-        self.shared_up_weight = self.shared_down_weight = None
+        self.shared_up_weight = self.shared_gate_up_weight = self.shared_down_weight = None
 
     def param_specs(self):
         E, f, hid = self.num_experts, self.inner_size, self.hidden_size
         specs = [ParamSpec("gate_up_weight", (E * 2 * f, hid)) if self.gated else ParamSpec("up_weight", (E * f, hid)),
                  ParamSpec("down_weight", (E * hid, f))]
-        if self.shared_inner:
+        if self.gated_shared:
+            specs += [ParamSpec("shared_gate_up_weight", (2 * self.shared_inner, hid)),
+                      ParamSpec("shared_down_weight", (hid, self.shared_inner))]
+        elif self.shared_inner:
             specs += [ParamSpec("shared_up_weight", (self.shared_inner, hid)),
                       ParamSpec("shared_down_weight", (hid, self.shared_inner)), ParamSpec("shared_gate_weight", (1, hid))]
         if self.routing == "table":
@@ -148,7 +159,14 @@ class MixtureOfExperts(Part):
         t = dict(tensors)
         if not self.gated:
             t["gate_up_weight"] = t.pop("up_weight")
-        if self.shared_inner:
+        if self.gated_shared:
+            pad, f = self.shared_padded - self.shared_inner, self.shared_inner
+            if pad:  # units of zero weight: every gate function maps (0, 0) to 0
+                fill = torch.nn.functional.pad
+                gu = t["shared_gate_up_weight"]
+                t["shared_gate_up_weight"] = torch.cat([fill(gu[:f], (0, 0, 0, pad)), fill(gu[f:], (0, 0, 0, pad))]).contiguous()
+                t["shared_down_weight"] = fill(t["shared_down_weight"], (0, pad)).contiguous()
+        elif self.shared_inner:
             # the shared feed-forward's gate is one more row of the router; rows up to a multiple of 8 are zero
             rows = [t["router_weight"], t.pop("shared_gate_weight")]
             fill = -(self.num_experts + 1) % 8
@@ -207,7 +225,7 @@ class MixtureOfExperts(Part):
         K.linear(h, self.router_weight, None, full)
         z = full[:, :E]
         choice = dict(top=top, group_count=self.group_count, group_keep=self.group_keep, score=self.score, ids=ids,
-                      weights=weights)
+                      weights=weights, weight_scale=self.weight_scale)
         if n <= K.MOE_ROUTE_FUSED_UP_TO and n * top <= K.MOE_TABLE_ROUTE_MAX_PAIRS:
             K.moe_select_route(z, self.correction, offsets=offsets, tiles=tiles, meta=meta, row_token=row_token,
                                place_of=place_of, place_weight=by_place, **choice)
@@ -217,7 +235,7 @@ class MixtureOfExperts(Part):
             K.moe_select(z, self.correction, counts=counts, **choice)
             K.moe_plan(ids, counts, fill, offsets, tiles, meta, row_token, place_of, n_tokens=n, n_experts=E, top=top,
                        weights=weights if self.weight_input else None, place_weight=by_place)
-        return weights, tiles, meta, row_token, place_of, by_place, full[:, E] if self.shared_inner else None
+        return weights, tiles, meta, row_token, place_of, by_place, full[:, E] if self.shared_inner and not self.gated else None
 
     def _experts(self, ctx, h, x, add: bool):
         """The experts' outputs, summed into ``x``, or (``x`` ``None``) left unsummed as a ``K.ExpertSum``."""
@@ -232,7 +250,13 @@ class MixtureOfExperts(Part):
             weights = None
         if self.shared_inner:
             u = ws.get("moe_shared_inner", (n, self.shared_padded), ctx.act_dtype)
-            K.linear(h, self.shared_up_weight, None, u, act=self.shared_act)
+            if self.gated_shared:
+                gu = ws.get("moe_shared_gate_up", (n, 2 * self.shared_padded), ctx.act_dtype)
+                K.linear(h, self.shared_gate_up_weight, None, gu)
+                K.gated_act(gu, u, width=self.shared_padded, up_at=self.shared_padded, gate=self.gate, alpha=self.alpha,
+                            limit=self.limit)
+            else:
+                K.linear(h, self.shared_up_weight, None, u, act=self.shared_act)
             shared = ws.get("moe_shared_out", (n, hid), torch.float32)
             K.linear(u, self.shared_down_weight, None, shared)
         act = ws.get("moe_inner", (n * top, f), ctx.act_dtype)

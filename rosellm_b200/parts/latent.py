@@ -9,8 +9,11 @@ values are linear in ``c``, the engine never expands them: the query takes ``W_u
 (csrc/latent_attention.cu), and ``W_uv`` is applied to the weighted sum of latents.  The cost of
 a decoded token is then one pass over ``kv_rank + rot_dim`` numbers per cached token for all
 heads together.  A softmax sink per head is optional; so are a latent for the queries (``q_rank``: ``c_q =
-norm(W_dq h)``, ``q = W_uq c_q``), an element-wise output gate on the merged heads (``gate``: times ``sigmoid(W_g
-h)``) and stretched rotation frequencies (``rot_scaling``).  Everything that multiplies the layer's input but
+norm(W_dq h)``, ``q = W_uq c_q``), an output gate on the heads' results (``gate``: ``"element"``, the merged heads times
+``sigmoid(W_g h)``; ``"head"``, head h's result times ``sigmoid((W_g h)_h)``), stretched rotation frequencies
+(``rot_scaling``), the pairs of a rotation (``rot_pairs``: ``"neighbours"``, entry 2i with 2i + 1, or ``"halves"``, entry
+i with i + dims/2) and rows taken from another layer's cache (``own_kv=False``: the layer has no ``W_dkv``; its runs carry
+``cache_of``).  Everything that multiplies the layer's input but
 feeds float32 arithmetic (the key/value latent, the query latent, the gate) is one product with float32 output.
 """
 from __future__ import annotations
@@ -30,7 +33,8 @@ class LatentAttention(Part):
 
     def __init__(self, hidden_size: int, num_heads: int, plain_dim: int, rot_dim: int, value_dim: int, kv_rank: int,
                  scale: float, rot_dims: int, rot_base: float, norm_eps: float, sink: bool = True,
-                 q_rank: int | None = None, gate: bool = False, rot_scaling: dict | None = None) -> None:
+                 q_rank: int | None = None, gate: str | None = None, rot_scaling: dict | None = None,
+                 rot_pairs: str = "neighbours", own_kv: bool = True) -> None:
         if min(hidden_size, num_heads, plain_dim, value_dim, kv_rank) <= 0 or rot_dim < 0:
             raise ValueError("latent attention: sizes must be positive")
         if hidden_size % 8:
@@ -45,7 +49,12 @@ class LatentAttention(Part):
         self.rotary = RotaryPositions(dims=rot_dims, base=rot_base, scaling=rot_scaling)
         if q_rank is not None and q_rank <= 0:
             raise ValueError("latent attention: the queries' latent must have a positive size")
-        self.q_rank, self.has_gate = q_rank, bool(gate)
+        if gate not in (None, "element", "head"):
+            raise ValueError(f"latent attention: gate {gate!r}; None, 'element' or 'head'")
+        if rot_pairs not in ("neighbours", "halves"):
+            raise ValueError(f"latent attention: rotation pairs {rot_pairs!r}; 'neighbours' or 'halves'")
+        self.q_rank, self.gate_kind, self.rot_pairs, self.own_kv = q_rank, gate, rot_pairs, bool(own_kv)
+        self.gate_width = {None: 0, "element": num_heads * value_dim, "head": num_heads}[gate]
         self.q_rank_padded = 0 if q_rank is None else -(-q_rank // 8) * 8
         # a cached row: the latent, the rotated part, zeros up to a multiple of 8 entries
         self.row_width = -(-(kv_rank + rot_dim) // 8) * 8
@@ -60,28 +69,45 @@ class LatentAttention(Part):
     def param_specs(self):
         H, hid = self.num_heads, self.hidden_size
         specs = [ParamSpec("q_weight", (H * self.head_in, hid if self.q_rank is None else self.q_rank)),
-                 ParamSpec("dkv_weight", (self.kv_rank + self.rot_dim, hid)),
-                 ParamSpec("dkv_norm", (self.kv_rank,), kind="vector", init="ones"),
                  ParamSpec("uk_weight", (H * self.plain_dim, self.kv_rank)),
                  ParamSpec("uv_weight", (H * self.value_dim, self.kv_rank)),
                  ParamSpec("o_weight", (hid, self.heads_width))]
+        if self.own_kv:
+            specs[1:1] = [ParamSpec("dkv_weight", (self.kv_rank + self.rot_dim, hid)),
+                          ParamSpec("dkv_norm", (self.kv_rank,), kind="vector", init="ones")]
         if self.has_sink:
             specs.append(ParamSpec("sink", (H,), kind="vector"))
         if self.q_rank is not None:
             specs += [ParamSpec("dq_weight", (self.q_rank, hid)),
                       ParamSpec("dq_norm", (self.q_rank,), kind="vector", init="ones")]
-        if self.has_gate:
-            specs.append(ParamSpec("gate_weight", (self.heads_width, hid)))
+        if self.gate_kind is not None:
+            specs.append(ParamSpec("gate_weight", (self.gate_width, hid)))
         return specs
+
+    def _neighbours(self, weight, first: int, period: int):
+        """The rows of ``weight`` with the turned entries of every rotated part (``period`` rows a part, beginning at row
+        ``first`` of each) brought from pairs (i, i + dims/2) to pairs (2i, 2i + 1), which the kernels turn.  Queries and
+        cached rows are reordered alike, so their products are what they were."""
+        n = self.rotary.dims // 2
+        if self.rot_pairs == "neighbours" or n == 0:
+            return weight
+        order = torch.arange(weight.shape[0])
+        for at in range(first, weight.shape[0], period):
+            turned = order[at:at + 2 * n].clone()
+            order[at:at + 2 * n:2], order[at + 1:at + 2 * n:2] = turned[:n], turned[n:]
+        return weight[order.to(weight.device)].contiguous()
 
     def bind(self, tensors) -> None:
         t = dict(tensors)
         dq, gate = t.pop("dq_weight", None), t.pop("gate_weight", None)
+        t["q_weight"] = self._neighbours(t["q_weight"], self.plain_dim, self.head_in)
+        if self.own_kv:
+            t["dkv_weight"] = self._neighbours(t["dkv_weight"], self.kv_rank, self.kv_rank + self.rot_dim)
         super().bind(t)
         # one product for all that multiplies the layer's input and is wanted in float32
-        names = (["dq"] if dq is not None else []) + ["dkv"] + (["g"] if gate is not None else [])
-        self.proj_weight, offs = pack_rows([{"dq": dq, "dkv": self.dkv_weight, "g": gate}[k] for k in names])
-        self.offsets = dict(zip(names, offs))
+        parts = {n: w for n, w in (("dq", dq), ("dkv", self.dkv_weight), ("g", gate)) if w is not None}
+        self.proj_weight, offs = pack_rows(list(parts.values())) if parts else (None, [])
+        self.offsets = dict(zip(parts, offs))
         self.dkv_weight = None  # it lives in the packed weight
         if self.q_rank is not None and self.q_rank_padded != self.q_rank:  # the product with W_uq reads 16-byte pieces
             self.q_weight = torch.nn.functional.pad(self.q_weight, (0, self.q_rank_padded - self.q_rank)).contiguous()
@@ -119,7 +145,9 @@ class LatentAttention(Part):
         table = ctx.block_table(run.cache_key)
         q = ws.get("latent_q", (n, H * self.head_in), act)
         off, proj = self.offsets, None
-        if run.writes_cache or len(off) > 1:
+        if run.writes_cache and not self.own_kv:
+            raise ValueError("latent attention: a layer without a key/value latent of its own reads another layer's cache")
+        if run.writes_cache or set(off) - {"dkv"}:
             proj = ws.get("latent_proj", (n, self.proj_weight.shape[0]), torch.float32)
             K.linear(h, self.proj_weight, None, proj)
         if self.q_rank is None:
@@ -161,9 +189,10 @@ class LatentAttention(Part):
             o = ws.get_zeroed(f"latent_heads_{self.heads_width}", (n, self.heads_padded), act)
         else:
             o = ws.get("latent_heads", (n, self.heads_padded), act)
-        gate, gate_strides = None, (0, 0)
-        if self.has_gate:  # the merged heads' gate rides on the product that makes them
-            gate, gate_strides = proj[:, off["g"]:off["g"] + self.heads_width], (proj.stride(0), self.value_dim)
+        gate, gate_strides = None, (0, 0, 1)
+        if self.gate_kind is not None:  # the gate rides on the product that makes the merged heads
+            gate = proj[:, off["g"]:off["g"] + self.gate_width]
+            gate_strides = (proj.stride(0), self.value_dim, 1) if self.gate_kind == "element" else (proj.stride(0), 1, 0)
         K.head_linear(o_lat, self.uv_weight, o, n_tokens=n, n_heads=H, k=rank, n=self.value_dim,
                       in_strides=(H * rank, rank), w_strides=(self.value_dim * rank, 1, rank),
                       out_strides=(self.heads_padded, self.value_dim), gate=gate, gate_strides=gate_strides)

@@ -1,6 +1,6 @@
 """Mixers that keep a matrix-valued state per request and head instead of a cache of keys.
 
-Both forms run one recurrence, ``S_t = diag(w_t) S_(t-1) [- (a_t * u_t)(u_t^T S_(t-1))] + k_t v_t^T`` and
+All but the last run one recurrence, ``S_t = diag(w_t) S_(t-1) [- (a_t * u_t)(u_t^T S_(t-1))] + k_t v_t^T`` and
 ``o_t = S_t^T r_t``, on the kernels of csrc/recurrent.cu: the state is float32 ``[heads, key size, value
 size]`` in the request's state slot (zero when the slot is taken), a step continues it for however many
 tokens the request brings, and everything between the projections and the output product is float32.
@@ -8,6 +8,9 @@ tokens the request brings, and everything between the projections and the output
 All projections of the layer's input are one product: the weights are packed at bind time (each
 tensor's rows filled up to a multiple of 8) and the product writes float32, so the recurrence reads
 unrounded projections in both precisions.
+
+``LightningAttention`` decays by a factor that does not depend on the token, so its portions of prompts are worked out
+chunk by chunk in parallel instead of token by token (csrc/lightning.cu).
 """
 from __future__ import annotations
 
@@ -288,4 +291,71 @@ class MatrixMemory(_StateMixer):
                      ctx.q_start, ctx.slots, prep, oraw, n_reqs=ctx.n_reqs, n_heads=self.num_heads, dk=self.key_dim,
                      dv=self.value_dim, eps=self.norm_eps, a_bias=self.i_bias, w0=self.f_bias, out_weight=self.out_norm,
                      cap=self.gate_cap, floor_eps=self.floor_eps, qscale=self.query_scale, gates=gates)
+        K.linear(buf, self.out_weight, None, x, residual=add)
+
+
+@register_part("mixer", "lightning_attention")
+class LightningAttention(_StateMixer):
+    """Linear attention whose state decays by one fixed factor a head.  ``q = silu(W_q h)``, ``k = silu(W_k h)`` (heads x
+    key_dim), ``v = silu(W_v h)`` (heads x value_dim; ``silu`` off: the projections as they come);
+    ``S_t = decay_h S_(t-1) + k_t v_t^T``, ``o_t = S_t^T q_t``.  The merged heads are divided by their common root mean
+    square over heads * value_dim (``norm_eps``), multiplied by ``out_norm`` (one entry per head and column) and by
+    ``sigmoid(W_g h)``, then ``W_o``.  ``decay``: a factor of [0, 1] per head.
+
+    Single tokens take one kernel that reads and writes the state once; portions take three (what each chunk of 64
+    tokens adds, the states between them, the outputs), in bfloat16 mode on the tensor cores (``tensor_cores``: ``None``
+    follows the activation type)."""
+
+    takes_projection = True  # forward(.., proj=): the input times ``proj_weight``, made by the caller
+
+    def __init__(self, hidden_size: int, num_heads: int, key_dim: int, value_dim: int, decay, norm_eps: float,
+                 silu: bool = True, tensor_cores: bool | None = None) -> None:
+        if key_dim > 256 or value_dim > 256:
+            raise ValueError(f"lightning attention: sizes {key_dim} / {value_dim}: the state kernels take up to 256")
+        decay = tuple(float(d) for d in decay)
+        if len(decay) != num_heads or not all(0.0 <= d <= 1.0 for d in decay):
+            raise ValueError(f"lightning attention: a decay between 0 and 1 for each of {num_heads} heads, got {decay}")
+        self.hidden_size, self.num_heads, self.key_dim, self.value_dim = hidden_size, num_heads, key_dim, value_dim
+        self.decay, self.norm_eps, self.silu, self.tensor_cores = decay, float(norm_eps), bool(silu), tensor_cores
+        self.key_width, self.out_width = num_heads * key_dim, num_heads * value_dim
+        self.out_padded = -(-self.out_width // 8) * 8
+        self.proj_weight = self.out_weight = self.out_norm = self._powers = None
+
+    def param_specs(self):
+        kw, vw, hid = self.key_width, self.out_width, self.hidden_size
+        return [ParamSpec("q_weight", (kw, hid)), ParamSpec("k_weight", (kw, hid)), ParamSpec("v_weight", (vw, hid)),
+                ParamSpec("g_weight", (vw, hid)), ParamSpec("out_norm", (vw,), kind="vector", init="ones"),
+                ParamSpec("out_weight", (hid, vw))]
+
+    def state_spec(self):
+        return StateSpec((self.num_heads, self.key_dim, self.value_dim), torch.float32)
+
+    def decay_powers(self) -> torch.Tensor:
+        """[heads, chunk + 1]: every head's decay to the powers 0 .. chunk (0^0 = 1), worked out in float64."""
+        d = torch.tensor(self.decay, dtype=torch.float64).view(-1, 1)
+        return torch.pow(d, torch.arange(K.LIGHTNING_CHUNK + 1, dtype=torch.float64)).to(torch.float32)
+
+    def bind(self, tensors) -> None:
+        t = dict(tensors)
+        names = ("q", "k", "v", "g")
+        self.proj_weight, offs = pack_rows([t[n + "_weight"] for n in names])
+        self.offsets = dict(zip(names, offs))
+        self.out_norm, self.out_weight = t["out_norm"], t["out_weight"]
+        self._powers = self.decay_powers().to(self.proj_weight.device)
+        self._pad_out_weight()
+
+    def forward(self, ctx, run, h, x, add: bool = True, proj=None) -> None:
+        proj = self._project(ctx, h, proj)
+        buf, view = self._out_buffer(ctx)
+        H, dk, dv, ws = self.num_heads, self.key_dim, self.value_dim, ctx.workspace
+        chunks = None
+        if ctx.n_tiles_wide:
+            chunks = ws.get("lightning_chunks", (ctx.n_tiles_wide * H * dk * dv,), torch.float32)
+        raw = ws.get("state_mixer_raw", (ctx.n_tokens, H * dv), torch.float32)
+        cores = ctx.act_dtype == torch.bfloat16 if self.tensor_cores is None else self.tensor_cores
+        K.lightning(proj, self.offsets, self._powers, ctx.state(run.state_key), ctx.q_start, ctx.slots, chunks, raw,
+                    n_heads=H, dk=dk, dv=dv, tiles=ctx.tiles_wide, n_tiles=ctx.n_tiles_wide, decode_reqs=ctx.decode_reqs,
+                    n_decode=ctx.n_decode, silu=self.silu, tensor_cores=cores)
+        g = self.offsets["g"]
+        K.rmsnorm_gate(raw, proj[:, g:g + self.out_width], self.out_norm, self.norm_eps, buf if view is None else view)
         K.linear(buf, self.out_weight, None, x, residual=add)

@@ -718,12 +718,16 @@ class PrePostNormBlock(Part):
 @register_part("head", "tied_to_embedding")
 class TiedHead(Part):
     """``logits = h wte^T`` with the embedding's own table, no bias
-    (rosellm/rosetrainer/model.py:503-504, 639-641)."""
+    (rosellm/rosetrainer/model.py:503-504, 639-641).  ``soft_cap``: the logits are bounded smoothly, ``soft_cap *
+    tanh(logits / soft_cap)``; where the head chooses the tokens itself, in its product's epilogue."""
 
     graph_safe = True
     launches_replayable = True
 
-    def __init__(self, vocab_size: int, hidden_size: int) -> None:
+    def __init__(self, vocab_size: int, hidden_size: int, soft_cap: float | None = None) -> None:
+        if soft_cap is not None and not soft_cap > 0:
+            raise ValueError(f"head: a bound of the logits must be positive, got {soft_cap}")
+        self.soft_cap = 0.0 if soft_cap is None else float(soft_cap)
         self.vocab_size = vocab_size
         self.hidden_size = hidden_size
         self.weight = None  # set by the model to the embedding's table
@@ -735,6 +739,8 @@ class TiedHead(Part):
         n_rows = h.x.shape[0] if isinstance(h, K.NormInput) else h.shape[0]
         logits = ctx.workspace.get("logits", (n_rows, self.vocab_size), torch.float32)
         K.linear(h, self.weight, None, logits)
+        if self.soft_cap:
+            K.soft_cap(logits, self.soft_cap)
         return logits
 
     def can_sample(self, n_rows: int, dtype: torch.dtype, with_temperature: bool = False) -> bool:
@@ -747,7 +753,7 @@ class TiedHead(Part):
         """The next token of every row of ``h`` into ``into.out_ids`` (arg-max, or by the rows'
         temperatures), chosen in the product's epilogue: what the sampling kernel would choose
         from ``forward``'s logits."""
-        K.linear_sample(h, self.weight, None, into)
+        K.linear_sample(h, self.weight, None, into, soft_cap=self.soft_cap)
 
 
 @register_part("head", "linear")
