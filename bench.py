@@ -71,6 +71,11 @@ def parse_args():
                    help="instead of the default workload: prefill and decode of the Vebotar design (differential attention "
                         "over chunks, a stream of two copies, routed experts beside a shared one) and of Soporax's windowed "
                         "attention and experts at equal width, depth and vocabulary")
+    p.add_argument("--compare-kugadra", action="store_true",
+                   help="instead of the default workload: prefill and decode of the Kugadra design (linear attention with a "
+                        "fixed decay per head, latent attention whose rows layers share, routed experts beside a shared one) "
+                        "beside Soporax's latent attention with experts and Fikevik's linear attention with decaying keys, "
+                        "at equal width, depth, vocabulary and projection sizes, random weights")
     p.add_argument("--compare-lebedra", action="store_true",
                    help="instead of the default workload: prefill and decode of the Lebedra design (latent attention, "
                         "mixture of experts) beside GPT-2 of equal width, depth and vocabulary, at layer sizes of "
@@ -959,6 +964,96 @@ def compare_vebotar(args):
     return 0
 
 
+# Layer sizes for --compare-kugadra: width; the linear attention's heads, key and value size; the latent attention's
+# heads, plain / turned / value size a head, its key/value latent and query latent; the dense inner size; experts,
+# experts a token, their inner size and the shared expert's.
+KUGADRA_SIZES = {
+    "1024": dict(width=1024, heads=8, dim=64, vdim=128, l_heads=16, l_dim=64, l_rot=32, l_vdim=64, kv_rank=256, q_rank=384,
+                 ff=4096, experts=16, top=2, expert_ff=1024, shared_ff=1024),
+    "2048": dict(width=2048, heads=16, dim=64, vdim=128, l_heads=16, l_dim=128, l_rot=64, l_vdim=128, kv_rank=512, q_rank=768,
+                 ff=8192, experts=32, top=4, expert_ff=1408, shared_ff=1408),
+}
+
+
+def _latent_mixer(z: dict) -> dict:
+    return {"heads": z["l_heads"], "dim": z["l_dim"], "rot_dim": z["l_rot"], "vdim": z["l_vdim"], "kv_rank": z["kv_rank"],
+            "q_rank": z["q_rank"], "scale": (z["l_dim"] + z["l_rot"]) ** -0.5,
+            "rot": {"dims": z["l_rot"], "base": 10000.0, "scaling": {"factor": 8.0, "original": 256, "fast": 16.0, "slow": 2.0}}}
+
+
+def kugadra_config(z: dict, layers: int, vocab: int, positions: int):
+    """Linear and latent attention in turn, the first layer with the dense feed-forward, the others with experts; every
+    second latent layer reads the rows of the one before it."""
+    from rosellm_b200.config.kugadra import KugadraConfig
+
+    lin = {"heads": z["heads"], "dim": z["dim"], "vdim": z["vdim"], "decay": [1.0 - 2.0 ** -(2 + i * 6.0 / z["heads"]) for i in range(z["heads"])]}
+    lat = _latent_mixer(z)
+    moe = {"kind": "moe", "expert": {"ff": z["expert_ff"]}, "router": {"experts": z["experts"], "top": z["top"], "scale": 2.5},
+           "shared": {"ff": z["shared_ff"]}}
+    out = []
+    for i in range(layers):
+        mixer = lin if i % 2 == 0 else (dict(lat, kv_from=i - 2) if i % 4 == 3 else lat)
+        out.append({"type": "lightning" if i % 2 == 0 else "latent_attention", "mixer": mixer,
+                    "mlp": {"kind": "dense", "ff": z["ff"]} if i == 0 else moe})
+    return KugadraConfig.from_dict({
+        "architecture": "Kugadra", "vocab": vocab, "width": z["width"], "max_positions": positions, "norm": {"eps": 1e-5},
+        "embedding": {"scale": float(z["width"]) ** 0.5}, "logit_softcap": 30.0, "layers": out})
+
+
+def kugadra_neighbours(z: dict, layers: int, vocab: int, positions: int):
+    """Soporax with latent attention of the same sizes in every layer, dense and expert feed-forwards as Kugadra's without
+    the shared expert; Fikevik with linear attention of the same sizes in every layer and dense feed-forwards."""
+    from rosellm_b200.config.fikevik import FikevikConfig
+    from rosellm_b200.config.soporax import SoporaxConfig
+
+    moe = {"kind": "moe", "expert": {"ff": z["expert_ff"]}, "router": {"experts": z["experts"], "top": z["top"]}}
+    soporax = SoporaxConfig.from_dict({
+        "architecture": "Soporax", "vocab": vocab, "width": z["width"], "max_positions": positions, "norm": {"eps": 1e-5},
+        "logit_scale": 0.5, "layers": [{"type": "latent_attention", "mixer": _latent_mixer(z),
+                                        "mlp": {"kind": "dense", "ff": z["ff"], "limit": 7.0} if i == 0 else moe}
+                                       for i in range(layers)]})
+    fikevik = FikevikConfig.from_dict({
+        "architecture": "Fikevik", "vocab": vocab, "width": z["width"], "max_positions": positions, "norm": {"eps": 1e-5},
+        "embedding": {"scale": float(z["width"]) ** 0.5}, "postln_alpha": 1.5,
+        "layers": [{"type": "gla", "mixer": {"heads": z["heads"], "dim": z["dim"], "vdim": z["vdim"], "tau": 16.0, "decay_rank": 16},
+                    "mlp": {"kind": "dense", "ff": z["ff"]}} for _ in range(layers)]})
+    return (("soporax", soporax), ("fikevik", fikevik))
+
+
+def compare_kugadra(args):
+    """Prefill (2 x 1024 tokens) and decode (batch 8 and 64, 512 cached tokens) of Kugadra and of the two shipped designs
+    that its mixers are nearest to: device time by CUDA events, as the default workload."""
+    layers, vocab, positions = 6, 32000, 1024
+    clocks = Clocks()
+    clocks.start()
+    out = {"metric": "prefill and decode of Kugadra beside Soporax's latent attention and Fikevik's linear attention at equal width",
+           "unit": "tokens/s", "n_gpus": 1,
+           "steps": args.steps, "warmup": args.warmup, "dtype": "bf16" if args.dtype == "bfloat16" else "fp32",
+           "data": "synthetic (random token ids, random weights)", "layers": layers, "vocab": vocab, "sizes": {}}
+    for name, z in KUGADRA_SIZES.items():
+        row = {}
+        for label, cfg in (("kugadra", kugadra_config(z, layers, vocab, positions)), *kugadra_neighbours(z, layers, vocab, positions)):
+            h = Harness(cfg, args.dtype, 64, graphs=not args.no_graphs)
+            try:
+                pms = h.prefill()
+                rec = {"prefill_2x1024_ms": round(pms, 4), "prefill_tok_s": round(2048 / (pms * 1e-3), 1),
+                       "weight_mb": round(h.runner.model.weight_bytes() / 1e6, 1)}
+                for b in (8, 64):
+                    ms, launches, gms, _ = h.device_decode(b, args.context, max(16, args.steps // 2), max(4, args.warmup // 2))
+                    rec[f"decode_b{b}_ms"] = round(ms, 4)
+                    rec[f"decode_b{b}_tok_s"] = round(b / (ms * 1e-3), 1)
+                    rec[f"decode_b{b}_launches"] = launches
+                    if gms is not None:
+                        rec[f"decode_b{b}_graph_ms"] = round(gms, 4)
+                row[label] = rec
+            finally:
+                h.close()
+        out["sizes"][name] = row
+    out["clocks"] = clocks.stop()
+    print(json.dumps(out))
+    return 0
+
+
 def main():
     args = parse_args()
     if args.gpus != 1:
@@ -974,6 +1069,8 @@ def main():
         return compare_soporax(args)
     if args.compare_vebotar:
         return compare_vebotar(args)
+    if args.compare_kugadra:
+        return compare_kugadra(args)
     if args.impl == "reference":
         run_reference(args)
     else:

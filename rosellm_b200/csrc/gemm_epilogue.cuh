@@ -74,7 +74,9 @@ struct SampleArgs {
   int* host_ring;
   int ring_stride;
   unsigned int* ring_step;
-  float soft_cap;  // > 0: the logits are soft_cap * tanh(logit / soft_cap) before anything else
+  // > 0: a row with a temperature draws from soft_cap * tanh(logit / soft_cap); the arg-max needs no bound, which keeps
+  // the order of the logits
+  float soft_cap;
 };
 constexpr unsigned int SAMPLE_RING = 4;
 

@@ -207,11 +207,11 @@ __global__ __launch_bounds__(32 * MAX_WARPS) void gemm_rows_bulk_kernel(
 #pragma unroll
     for (int hlf = 0; hlf < 2; ++hlf) {
       const float temp = temp2[hlf];
-      float s0 = soft_capped(c[2 * hlf] + bias0, sample.soft_cap), s1 = soft_capped(c[2 * hlf + 1] + bias1, sample.soft_cap);
+      float s0 = c[2 * hlf] + bias0, s1 = c[2 * hlf + 1] + bias1;
       if (temp > 0.f) {
         const float inv_t = 1.0f / temp;
-        s0 = sample_key(s0, inv_t, seed2[hlf], counter2[hlf], (uint32_t)n);
-        s1 = sample_key(s1, inv_t, seed2[hlf], counter2[hlf], (uint32_t)(n + 1));
+        s0 = sample_key(soft_capped(s0, sample.soft_cap), inv_t, seed2[hlf], counter2[hlf], (uint32_t)n);
+        s1 = sample_key(soft_capped(s1, sample.soft_cap), inv_t, seed2[hlf], counter2[hlf], (uint32_t)(n + 1));
       }
       ArgMax& best = hlf ? best_hi : best_lo;
       if (n < N) best = better(best, ArgMax{s0, n});

@@ -352,14 +352,13 @@ __global__ __launch_bounds__(32 * KSPLIT * GROUPS) void gemm_rows_mma_kernel(
           const int m = t * 16 + hlf * 8 + g;
           const int mc = m < M ? m : 0;  // every lane takes part in the exchanges below
           const float temp = temp_of[t][hlf];
-          float s0 = soft_capped(apply_act(c[t][2 * hlf] + bias0, act), sample.soft_cap);
-          float s1 = soft_capped(apply_act(c[t][2 * hlf + 1] + bias1, act), sample.soft_cap);
+          float s0 = apply_act(c[t][2 * hlf] + bias0, act), s1 = apply_act(c[t][2 * hlf + 1] + bias1, act);
           if (temp > 0.f) {
             const uint64_t seed = (uint64_t)sample.seeds[mc];
             const uint32_t counter = (uint32_t)sample.counters[mc];
             const float inv_t = 1.0f / temp;
-            s0 = sample_key(s0, inv_t, seed, counter, (uint32_t)n);
-            s1 = sample_key(s1, inv_t, seed, counter, (uint32_t)(n + 1));
+            s0 = sample_key(soft_capped(s0, sample.soft_cap), inv_t, seed, counter, (uint32_t)n);
+            s1 = sample_key(soft_capped(s1, sample.soft_cap), inv_t, seed, counter, (uint32_t)(n + 1));
           }
           ArgMax best{-CUDART_INF_F, 0x7fffffff};
           if (n < N) best = ArgMax{s0, n};
@@ -583,8 +582,8 @@ RL_EXPORT int rl_gemm_rows_bf16(int out_dtype, const void* A, long lda, const vo
 // written: out_ids[m] is what rl_sample would choose from row m of A W^T (+ bias) with the same
 // temperature, seed and counter (rows with top-k or top-p are not for this entry point).
 // best [M] and ticket [1] are scratch that is zero before the call and zero again after it.
-// host_ring != nullptr: the ids are also written to that pinned host memory (see SampleArgs).  soft_cap > 0: the logits
-// are soft_cap * tanh(logit / soft_cap).
+// host_ring != nullptr: the ids are also written to that pinned host memory (see SampleArgs).  soft_cap > 0: rows with
+// a temperature draw from soft_cap * tanh(logit / soft_cap).
 RL_EXPORT int rl_gemm_rows_bf16_sample(const void* A, long lda, const void* W, const float* bias, int M, int N, int K,
                                        const float* norm_x, long norm_ldx, const float* norm_gamma,
                                        const float* norm_beta, float norm_eps, const float* temperature,

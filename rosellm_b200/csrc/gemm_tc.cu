@@ -65,11 +65,10 @@ __host__ __device__ constexpr int staging_bytes() {
 constexpr int BAR_BYTES = (2 * MAX_STAGES + 4) * 8 + 16;
 constexpr int SMEM_BUDGET = 227 * 1024;
 
-__device__ __noinline__ float sample_key_call(float logit, float inv_t, uint64_t seed, uint32_t counter, uint32_t index) {
-  return sample_key(logit, inv_t, seed, counter, index);
+__device__ __noinline__ float sample_key_call(float logit, float inv_t, uint64_t seed, uint32_t counter, uint32_t index,
+                                              float cap) {
+  return sample_key(soft_capped(logit, cap), inv_t, seed, counter, index);
 }
-
-__device__ __noinline__ float soft_capped_call(float v, float cap) { return soft_capped(v, cap); }
 
 // What a launch is told beyond the tensor maps.
 struct PArgs {
@@ -336,23 +335,20 @@ __global__ __launch_bounds__(PTHREADS, 1) void gemm_tc_persistent_kernel(const _
           asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
           const float bias_c = c == part ? bias0 : bias1;
           const int col0 = n0 + c * 32;
-          if (!any_sampled && sm.soft_cap <= 0.f) {
+          if (!any_sampled) {
 #pragma unroll
             for (int i = 0; i < 32; ++i) {
               const float v = act_fn(__uint_as_float(r[i]) + __shfl_sync(0xffffffffu, bias_c, i), p.act);
               if (col0 + i < N) best = better(best, ArgMax{v, col0 + i});
             }
           } else {
-            // noise and bound are calls, not thirty-two inlined copies: the loop of the rows that take
+            // the noise is a call, not thirty-two inlined copies: the loop of the rows that take
             // the arg-max (above) stays short, and so does what the instruction cache must hold
 #pragma unroll
             for (int i = 0; i < 32; ++i) {
               float v = act_fn(__uint_as_float(r[i]) + __shfl_sync(0xffffffffu, bias_c, i), p.act);
-              if (sm.soft_cap > 0.f) v = soft_capped_call(v, sm.soft_cap);
-              if (any_sampled) {
-                const float key = sample_key_call(v, inv_t, seed, counter, (uint32_t)(col0 + i));
-                if (temp > 0.f) v = key;
-              }
+              const float key = sample_key_call(v, inv_t, seed, counter, (uint32_t)(col0 + i), sm.soft_cap);
+              if (temp > 0.f) v = key;
               if (col0 + i < N) best = better(best, ArgMax{v, col0 + i});
             }
           }

@@ -130,7 +130,7 @@ __global__ __launch_bounds__(256) void lightning_out_simt_kernel(const Lightning
 // ---- the states between the chunks ------------------------------------------------------------------------------
 
 // Grid (tiles, heads, pieces of a head's state): the blocks of a portion's first tile walk its tiles, a thread VEC
-// elements of the state.  Four chunks are fetched ahead of the four that are used.
+// elements of the state, eight chunks' worth fetched at a time.
 template <int VEC>
 __global__ __launch_bounds__(256) void lightning_scan_kernel(const LightningParams p, const int* __restrict__ tiles) {
   pdl_begin();
@@ -161,7 +161,7 @@ __global__ __launch_bounds__(256) void lightning_scan_kernel(const LightningPara
     else *to = from[0];
   };
   get(st, S);
-  constexpr int AHEAD = 4;
+  constexpr int AHEAD = 8;
   for (int c0 = 0; c0 < n_chunks; c0 += AHEAD) {
     float x[AHEAD][VEC];
 #pragma unroll
@@ -196,12 +196,6 @@ __device__ __forceinline__ uint32_t pack2(float lo, float hi) {
   const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
   return *reinterpret_cast<const uint32_t*>(&v);
 }
-// x = hi + lo + (at most 2^-17 |x|)
-__device__ __forceinline__ void split_bf16(float x, __nv_bfloat16& hi, __nv_bfloat16& lo) {
-  hi = __float2bfloat16_rn(x);
-  lo = __float2bfloat16_rn(x - __bfloat162float(hi));
-}
-
 // `rows` x `cols` elements f(row, column) of a float32 matrix into a bfloat16 tile of 64 (or `rows_pad`) rows, zeros outside.
 // VEC: columns in fours, 16-byte loads.
 template <bool VEC, class Put>
@@ -230,6 +224,7 @@ __device__ __forceinline__ void store_bf16(__nv_bfloat16* dst, const float (&x)[
     dst[0] = __float2bfloat16_rn(x[0]);
   }
 }
+// x = hi + lo + (at most 2^-17 |x|)
 template <int W>
 __device__ __forceinline__ void store_split(__nv_bfloat16* hi, __nv_bfloat16* lo, const float (&x)[W]) {
   float rest[W];
@@ -258,7 +253,7 @@ __global__ __launch_bounds__(128) void lightning_chunk_mma_kernel(const Lightnin
   const float* row = p.proj + (size_t)t.tok * p.ldp;
   lightning_stage<VEC>(row + p.off_k + h * p.dk, p.ldp, t.n, p.dk, LG_C, dkp, [&](int r, int c, auto& x) {
     const float w = r < t.n ? pw_s[t.n - 1 - r] : 0.f;
-    for (auto& e : x) e = lightning_act_fast(e, p.act) * w;
+    for (auto& e : x) e = __bfloat162float(__float2bfloat16_rn(lightning_act_fast(e, p.act))) * w;  // the key as lightning_out_mma_kernel has it
     store_split(k_hi + r * LDK + c, k_lo + r * LDK + c, x);
   });
   lightning_stage<VEC>(row + p.off_v + h * p.dv + n0, p.ldp, t.n, p.dv - n0, LG_C, LG_N, [&](int r, int c, auto& x) {

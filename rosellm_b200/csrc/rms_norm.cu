@@ -122,6 +122,105 @@ __global__ __launch_bounds__(256) void rmsnorm_add_norm_kernel(const float* __re
   for (int d = threadIdx.x; d < width; d += blockDim.x) o[d] = from_f32<TOut>(row_s[d] * r2 * gamma_next[d]);
 }
 
+// What a sublayer gave, row by row: y itself, or (y null) a mixture of experts not yet summed: sum_j weights[t, j] *
+// eo[place_of[t, j]] + shared[t] * sigmoid(sg[t]) (weights, shared, sg may be null: factors of 1, nothing added), in
+// moe_combine_kernel's order.
+struct SublayerRows {
+  const float* y;
+  long ldy;
+  const float* eo;
+  const float* weights;
+  const int* place_of;
+  int top;
+  const float* shared;
+  long ldshared;
+  const float* sg;
+  long ldsg;
+};
+
+// The same two norms with everything a row needs in flight at once: a thread keeps its KEEP pieces of four entries of the
+// sublayer's row, the stream's row and both norms' weights in registers (the weights are fetched before the wait for the
+// kernels ahead), and the sum over a token's experts is formed on the way in (fused: no combine kernel, no buffer of
+// summed rows).  NEXT off: the addition to the stream alone.
+template <typename TOut, int KEEP, bool EXPERTS, bool NEXT>
+__global__ __launch_bounds__(256) void rmsnorm_add_norm_vec_kernel(const SublayerRows src, const float* __restrict__ gamma,
+                                                                   float* __restrict__ stream, long lds,
+                                                                   const float* __restrict__ gamma_next, TOut* __restrict__ next,
+                                                                   long ldn, int width, float eps, float eps_next) {
+  __shared__ float scratch[33];
+  const int i = blockIdx.x, pieces = width / 4;
+  float4 y[KEEP], x[KEEP], g[KEEP], gn[KEEP];
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+#pragma unroll
+  for (int k = 0; k < KEEP; ++k) {
+    const int d = threadIdx.x + k * blockDim.x;
+    g[k] = d < pieces ? reinterpret_cast<const float4*>(gamma)[d] : zero;
+    if (NEXT) gn[k] = d < pieces ? reinterpret_cast<const float4*>(gamma_next)[d] : zero;
+  }
+  asm volatile("griddepcontrol.wait;" ::: "memory");
+  float4* xr = reinterpret_cast<float4*>(stream + (size_t)i * lds);
+#pragma unroll
+  for (int k = 0; k < KEEP; ++k) {
+    const int d = threadIdx.x + k * blockDim.x;
+    x[k] = d < pieces ? xr[d] : zero;
+    if (EXPERTS) y[k] = zero;
+    else y[k] = d < pieces ? reinterpret_cast<const float4*>(src.y + (size_t)i * src.ldy)[d] : zero;
+  }
+  if (EXPERTS) {
+    auto add = [&](float w, const float* row) {
+#pragma unroll
+      for (int k = 0; k < KEEP; ++k) {
+        const int d = threadIdx.x + k * blockDim.x;
+        if (d < pieces) {
+          const float4 v = reinterpret_cast<const float4*>(row)[d];
+          y[k].x = fmaf(w, v.x, y[k].x);
+          y[k].y = fmaf(w, v.y, y[k].y);
+          y[k].z = fmaf(w, v.z, y[k].z);
+          y[k].w = fmaf(w, v.w, y[k].w);
+        }
+      }
+    };
+#pragma unroll 4
+    for (int j = 0; j < src.top; ++j) {
+      const size_t at = (size_t)i * src.top + j;
+      add(src.weights != nullptr ? src.weights[at] : 1.f, src.eo + (size_t)src.place_of[at] * width);
+    }
+    if (src.shared != nullptr)
+      add(src.sg != nullptr ? 1.0f / (1.0f + expf(-src.sg[(size_t)i * src.ldsg])) : 1.f, src.shared + (size_t)i * src.ldshared);
+  }
+  float s = 0.f;
+#pragma unroll
+  for (int k = 0; k < KEEP; ++k) s = fmaf(y[k].x, y[k].x, fmaf(y[k].y, y[k].y, fmaf(y[k].z, y[k].z, fmaf(y[k].w, y[k].w, s))));
+  const float r = 1.0f / sqrtf(block_sum(s, scratch) / (float)width + eps);
+  float s2 = 0.f;
+#pragma unroll
+  for (int k = 0; k < KEEP; ++k) {
+    const int d = threadIdx.x + k * blockDim.x;
+    x[k].x += y[k].x * r * g[k].x;
+    x[k].y += y[k].y * r * g[k].y;
+    x[k].z += y[k].z * r * g[k].z;
+    x[k].w += y[k].w * r * g[k].w;
+    if (d < pieces) xr[d] = x[k];
+    s2 = fmaf(x[k].x, x[k].x, fmaf(x[k].y, x[k].y, fmaf(x[k].z, x[k].z, fmaf(x[k].w, x[k].w, s2))));
+  }
+  if (!NEXT) return;
+  const float r2 = 1.0f / sqrtf(block_sum(s2, scratch) / (float)width + eps_next);
+  TOut* o = next + (size_t)i * ldn;
+#pragma unroll
+  for (int k = 0; k < KEEP; ++k) {
+    const int d = threadIdx.x + k * blockDim.x;
+    if (d >= pieces) continue;
+    const float4 v = make_float4(x[k].x * r2 * gn[k].x, x[k].y * r2 * gn[k].y, x[k].z * r2 * gn[k].z, x[k].w * r2 * gn[k].w);
+    if (sizeof(TOut) == 4) {
+      reinterpret_cast<float4*>(o)[d] = v;
+    } else {
+      const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+      reinterpret_cast<uint2*>(o)[d] = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+    }
+  }
+}
+
 __global__ void cast_rows_kernel(const float* __restrict__ x, __nv_bfloat16* __restrict__ out, long n) {
   pdl_begin();
   const long i = (long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -177,6 +276,20 @@ static inline int norm_threads(int width) {
   return t < 32 ? 32 : (t > 256 ? 256 : t);
 }
 
+constexpr int RMS_VEC_MAX_WIDTH = 4 * 4 * 256;  // four pieces of four entries for each of 256 threads
+
+template <typename TOut, bool EXPERTS, bool NEXT>
+static void launch_add_norm_vec(const SublayerRows& src, const float* gamma, float* stream_rows, long lds, const float* gamma_next,
+                                TOut* next, long ldn, int n_rows, int width, float eps, float eps_next, cudaStream_t stream) {
+  const int pieces = width / 4;
+  int threads = (pieces + 31) / 32 * 32;
+  threads = threads > 256 ? 256 : threads;
+  auto kernel = pieces <= threads ? rmsnorm_add_norm_vec_kernel<TOut, 1, EXPERTS, NEXT>
+                                  : (pieces <= 2 * threads ? rmsnorm_add_norm_vec_kernel<TOut, 2, EXPERTS, NEXT>
+                                                           : rmsnorm_add_norm_vec_kernel<TOut, 4, EXPERTS, NEXT>);
+  launch_pdl(kernel, n_rows, threads, 0, stream, src, gamma, stream_rows, lds, gamma_next, next, ldn, width, eps, eps_next);
+}
+
 }  // namespace rl
 
 // out[i] = rmsnorm(x[rows[i]] or x[i]) * gamma.  out_dtype: RL_F32 or RL_BF16.
@@ -222,6 +335,20 @@ RL_EXPORT int rl_rmsnorm_add_norm(int out_dtype, const float* y, long ldy, const
                                   float eps, float eps_next, cudaStream_t stream) {
   if (n_rows <= 0) return 0;
   if (width <= 0 || width > 48 * 1024 / 4 - 64) return -2;
+  const int osize = out_dtype == RL_F32 ? 4 : 2;
+  if (width % 4 == 0 && width <= rl::RMS_VEC_MAX_WIDTH && ldy % 4 == 0 && lds % 4 == 0 && ldn % 4 == 0 && (uintptr_t)y % 16 == 0 &&
+      (uintptr_t)stream_rows % 16 == 0 && (uintptr_t)gamma % 16 == 0 && (uintptr_t)gamma_next % 16 == 0 &&
+      (uintptr_t)next % (4 * osize) == 0) {
+    const rl::SublayerRows src{y, ldy};
+    if (out_dtype == RL_F32)
+      rl::launch_add_norm_vec<float, false, true>(src, gamma, stream_rows, lds, gamma_next, (float*)next, ldn, n_rows, width, eps,
+                                                  eps_next, stream);
+    else
+      rl::launch_add_norm_vec<__nv_bfloat16, false, true>(src, gamma, stream_rows, lds, gamma_next, (__nv_bfloat16*)next, ldn, n_rows,
+                                                          width, eps, eps_next, stream);
+    RL_CHECK_LAUNCH();
+    return 0;
+  }
   const size_t smem = (size_t)(width + 33) * sizeof(float);
   if (out_dtype == RL_F32)
     rl::launch_pdl(rl::rmsnorm_add_norm_kernel<float>, n_rows, rl::norm_threads(width), smem, stream, y, ldy, gamma,
@@ -229,6 +356,36 @@ RL_EXPORT int rl_rmsnorm_add_norm(int out_dtype, const float* y, long ldy, const
   else
     rl::launch_pdl(rl::rmsnorm_add_norm_kernel<__nv_bfloat16>, n_rows, rl::norm_threads(width), smem, stream, y, ldy,
                    gamma, stream_rows, lds, gamma_next, (__nv_bfloat16*)next, ldn, n_rows, width, eps, eps_next);
+  RL_CHECK_LAUNCH();
+  return 0;
+}
+
+// 1 if rl_rmsnorm_add_experts takes rows of this width.
+RL_EXPORT int rl_rmsnorm_add_experts_fits(int width) { return width > 0 && width % 4 == 0 && width <= rl::RMS_VEC_MAX_WIDTH; }
+
+// The same (next null: without the second norm) for a mixture of experts not yet summed: y[t] = sum_j weights[t, j] *
+// eo[place_of[t, j]] + shared[t] * sigmoid(sg[t]); eo float32 [pairs, width], the rest as rl_moe_experts takes it.  Rows in
+// 16-byte pieces.
+RL_EXPORT int rl_rmsnorm_add_experts(int out_dtype, const float* eo, const float* weights, const int* place_of, int top,
+                                     const float* shared, long ldshared, const float* sg, long ldsg, const float* gamma,
+                                     float* stream_rows, long lds, const float* gamma_next, void* next, long ldn, int n_rows,
+                                     int width, float eps, float eps_next, cudaStream_t stream) {
+  if (n_rows <= 0) return 0;
+  const int osize = out_dtype == RL_F32 ? 4 : 2;
+  if (!rl_rmsnorm_add_experts_fits(width) || top <= 0 || (shared == nullptr && sg != nullptr) || (next != nullptr && gamma_next == nullptr) ||
+      ldshared % 4 != 0 || lds % 4 != 0 || ldn % 4 != 0 ||
+      (((uintptr_t)eo | (uintptr_t)shared | (uintptr_t)gamma | (uintptr_t)gamma_next | (uintptr_t)stream_rows) % 16) != 0 ||
+      (uintptr_t)next % (4 * osize) != 0)
+    return -2;
+  const rl::SublayerRows src{nullptr, 0, eo, weights, place_of, top, shared, ldshared, sg, ldsg};
+  if (next == nullptr)
+    rl::launch_add_norm_vec<float, true, false>(src, gamma, stream_rows, lds, nullptr, nullptr, 0, n_rows, width, eps, eps_next, stream);
+  else if (out_dtype == RL_F32)
+    rl::launch_add_norm_vec<float, true, true>(src, gamma, stream_rows, lds, gamma_next, (float*)next, ldn, n_rows, width, eps,
+                                               eps_next, stream);
+  else
+    rl::launch_add_norm_vec<__nv_bfloat16, true, true>(src, gamma, stream_rows, lds, gamma_next, (__nv_bfloat16*)next, ldn, n_rows,
+                                                       width, eps, eps_next, stream);
   RL_CHECK_LAUNCH();
   return 0;
 }

@@ -94,7 +94,7 @@ class _RecordingLib:
 
 _QUERIES = ("rl_gemm_tc_rows_fits", "rl_gemm_rows_smem_fits", "rl_mlp_fused_slice", "rl_attn_block_fused_fits", "rl_attn_block_fused_cluster",
             "rl_host_memory_on_device", "rl_latent_attention_fits", "rl_latent_decode_fits",
-            "rl_moe_max_tiles", "rl_bias_attention_shape", "rl_recurrence_record")  # library functions that launch nothing
+            "rl_moe_max_tiles", "rl_bias_attention_shape", "rl_recurrence_record", "rl_rmsnorm_add_experts_fits")  # library functions that launch nothing
 
 
 class recording:
@@ -161,7 +161,7 @@ def _lib() -> ctypes.CDLL:
         lib.rl_latent_q_rope.argtypes = [I, P, L, I, I, P, L, I, I, I, I, P, P, I, I, F, P]
         lib.rl_latent_attention.argtypes = [I, P, L, P, P, I, P, P, P, P, L, P, I, I, I, I, F, P, I, P, I, I, I, P, P, I, P, P]
         lib.rl_head_linear.argtypes = [I, P, L, L, P, L, L, L, P, L, L, I, I, I, I, P, L, L, L, P]
-        lib.rl_gated_act.argtypes = [I, P, L, I, P, L, I, I, I, F, F, P]
+        lib.rl_gated_act.argtypes = [I, I, P, L, I, P, L, I, I, I, F, F, P]
         lib.rl_token_gate.argtypes = [I, P, L, P, P, L, I, I, P, L, I, I, I, P, I, P, P]
         lib.rl_moe_select.argtypes = [P, L, P, I, I, I, I, I, I, F, P, P, P, P]
         lib.rl_moe_plan.argtypes = [P, P, P, P, P, P, P, P, P, P, I, I, I, P]
@@ -171,6 +171,8 @@ def _lib() -> ctypes.CDLL:
         lib.rl_hyper_step.argtypes = [I, P, L, L, P, L, P, L, P, P, P, P, F, P, L, P, L, I, I, I, P, P, P, I, P, L, P, L, P]
         lib.rl_embed_pair.argtypes = [I, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, P, P, P, I, P]
         lib.rl_rmsnorm_add_norm.argtypes = [I, P, L, P, P, L, P, P, L, I, I, F, F, P]
+        lib.rl_rmsnorm_add_experts.argtypes = [I, P, P, P, I, P, L, P, L, P, P, L, P, P, L, I, I, F, F, P]
+        lib.rl_rmsnorm_add_experts_fits.argtypes = [I]
         lib.rl_recurrence.argtypes = [I, I, P, L, I, I, I, I, I, I, P, P, P, I, P, P, P, L, P, P, P, P, I, I, I, I, I, F, F, F,
                                       L, I, F, F, F, F, P, P]
         lib.rl_recurrence_record.argtypes = [I, I, I, P, P, P]
@@ -195,7 +197,8 @@ def _lib() -> ctypes.CDLL:
                      "rl_rmsnorm_add_norm", "rl_recurrence", "rl_recurrence_record", "rl_bias_attention_shape", "rl_bias_attention",
                      "rl_bias_kv_store", "rl_qkv_norm_rotate", "rl_gated_join_norm", "rl_stream_inject", "rl_gate_mul",
                      "rl_moe_table_select", "rl_stream_inject_norm", "rl_moe_table_route",
-                     "rl_moe_select_route", "rl_hyper_step", "rl_lightning", "rl_rmsnorm_gate", "rl_soft_cap"):
+                     "rl_moe_select_route", "rl_hyper_step", "rl_lightning", "rl_rmsnorm_gate", "rl_soft_cap",
+                     "rl_rmsnorm_add_experts", "rl_rmsnorm_add_experts_fits"):
             getattr(lib, name).restype = I
         for name in ("rl_copy_to_device", "rl_event_record", "rl_embed", "rl_layernorm", "rl_gemm_simt", "rl_gemm_tc", "rl_gemm_tc_sample", "rl_gemm_tc_cut", "rl_gemm_tc_rows", "rl_gemm_tc_rows_fits",
                      "rl_gemm_rows_smem", "rl_gemm_rows_smem_fits",
@@ -603,7 +606,8 @@ def linear_sample(a, weight, bias, into: SampleInto, soft_cap: float = 0.0) -> N
     (arg-max, or with a temperature the arg-max of logit / temperature + Gumbel noise), without
     the logits being written anywhere.  bfloat16, where ``sampling_product_possible``;
     ``a`` may be a ``NormInput`` as for ``linear``.  Rows with top-k or top-p need their logits:
-    they are not for this call.  ``soft_cap`` > 0: a logit is soft_cap * tanh(logit / soft_cap)."""
+    they are not for this call.  ``soft_cap`` > 0: rows with a temperature draw from soft_cap * tanh(logit / soft_cap)
+    (the arg-max is the same with and without)."""
     norm = a if isinstance(a, NormInput) else None
     _need(weight, "weight", torch.bfloat16)
     n, k = weight.shape
@@ -1121,12 +1125,13 @@ UNITS = {"relu_squared": 4}  # activations of layers with one input projection (
 
 
 def gated_act(gu, out, *, width: int, up_at: int, gate: int, alpha: float = 1.0, limit: float = 0.0) -> None:
-    """out[r, f] = f(gu[r, f], gu[r, up_at + f]) for f < width (see csrc/gated_act.cuh)."""
+    """out[r, f] = f(gu[r, f], gu[r, up_at + f]) for f < width (see csrc/gated_act.cuh); ``out`` of ``gu``'s dtype, or
+    bfloat16 from float32."""
     _need(gu, "gu", contiguous=False)
-    _need(out, "out", gu.dtype, contiguous=False)
-    if gu.shape[1] < up_at + width or out.shape[1] < width or out.shape[0] != gu.shape[0]:
+    _need(out, "out", contiguous=False)
+    if gu.shape[1] < up_at + width or out.shape[1] < width or out.shape[0] != gu.shape[0] or gu.stride(1) != 1 or out.stride(1) != 1:
         raise KernelError("gated_act: shapes do not fit")
-    _ok(_lib().rl_gated_act(_code(gu), _ptr(gu), gu.stride(0), up_at, _ptr(out), out.stride(0), gu.shape[0], width,
+    _ok(_lib().rl_gated_act(_code(gu), _code(out), _ptr(gu), gu.stride(0), up_at, _ptr(out), out.stride(0), gu.shape[0], width,
                             gate, float(alpha), float(limit), _stream()), "gated_act")
 
 
@@ -1468,6 +1473,38 @@ def rmsnorm_add_norm(y, gamma, eps: float, stream_rows, gamma_next, eps_next: fl
 
 
 RMSNORM_ADD_NORM_MAX_WIDTH = 48 * 1024 // 4 - 64
+
+
+def rmsnorm_add_experts_fits(width: int) -> bool:
+    """Whether ``rmsnorm_add_experts`` takes rows of this width."""
+    return bool(_lib().rl_rmsnorm_add_experts_fits(width))
+
+
+def rmsnorm_add_experts(y: "ExpertSum", gamma, eps: float, stream_rows, gamma_next=None, eps_next: float = 0.0, out_next=None) -> None:
+    """``rmsnorm_add_norm`` for a mixture of experts not yet summed (``y``): the sum over a token's experts, the norm, the
+    addition to the stream and (``out_next`` given) the norm ahead of the next sublayer in one pass."""
+    _need(gamma, "gamma", torch.float32)
+    _need(stream_rows, "stream_rows", torch.float32, contiguous=False)
+    n, width = stream_rows.shape
+    if y.eo.numel() < n * y.top * width or gamma.numel() != width or stream_rows.stride(1) != 1 or y.place_of.numel() < n * y.top \
+            or (y.weights is not None and y.weights.numel() < n * y.top):
+        raise KernelError("rmsnorm_add_experts: shapes differ")
+    if y.shared is not None and (tuple(y.shared.shape) != (n, width) or y.shared.stride(1) != 1):
+        raise KernelError("rmsnorm_add_experts: the shared feed-forward's output has another shape")
+    if out_next is not None:
+        _need(gamma_next, "gamma_next", torch.float32)
+        _need(out_next, "out_next", contiguous=False)
+        if tuple(out_next.shape) != (n, width) or gamma_next.numel() != width or out_next.stride(1) != 1:
+            raise KernelError("rmsnorm_add_experts: shapes differ")
+    rc = _lib().rl_rmsnorm_add_experts(F32 if out_next is None else _code(out_next), _ptr(y.eo), _ptr(y.weights), _ptr(y.place_of),
+                                       y.top, _ptr(y.shared), 0 if y.shared is None else y.shared.stride(0), _ptr(y.shared_gate),
+                                       0 if y.shared_gate is None else y.shared_gate.stride(0), _ptr(gamma), _ptr(stream_rows),
+                                       stream_rows.stride(0), _ptr(gamma_next) if out_next is not None else None, _ptr(out_next),
+                                       0 if out_next is None else out_next.stride(0), n, width, float(eps), float(eps_next),
+                                       _stream())
+    if rc == -2:
+        raise KernelError(f"rmsnorm_add_experts: rows of {width} entries, or operands that are not 16-byte aligned, not taken")
+    _ok(rc, "rmsnorm_add_experts")
 
 
 # ---- mixers with a matrix-valued state -------------------------------------------------------------

@@ -11,6 +11,7 @@ import torch
 
 from ..ops import kernels as K
 from .base import ParamSpec, Part, register_part
+from .recurrent import pack_rows
 
 
 def _gate(name: str) -> int:
@@ -135,7 +136,8 @@ class MixtureOfExperts(Part):
         self.gated_shared = bool(shared_inner) and self.gated
         self.has_correction = bool(correction)
         self.router_weight = self.correction = self.gate_up_weight = self.down_weight = self.table = None
-        self.shared_up_weight = self.shared_gate_up_weight = self.shared_down_weight = None
+        self.shared_up_weight = self.shared_down_weight = None
+        self.shared_at = 0  # first column of a gated shared feed-forward's projections in the router's product
 
     def param_specs(self):
         E, f, hid = self.num_experts, self.inner_size, self.hidden_size
@@ -161,11 +163,13 @@ class MixtureOfExperts(Part):
             t["gate_up_weight"] = t.pop("up_weight")
         if self.gated_shared:
             pad, f = self.shared_padded - self.shared_inner, self.shared_inner
-            if pad:  # units of zero weight: every gate function maps (0, 0) to 0
-                fill = torch.nn.functional.pad
-                gu = t["shared_gate_up_weight"]
-                t["shared_gate_up_weight"] = torch.cat([fill(gu[:f], (0, 0, 0, pad)), fill(gu[f:], (0, 0, 0, pad))]).contiguous()
-                t["shared_down_weight"] = fill(t["shared_down_weight"], (0, pad)).contiguous()
+            gu = t.pop("shared_gate_up_weight")
+            # one product for the router and the shared feed-forward's two projections: both read the layer's input
+            # (units between them, and those that fill its inner size up to a multiple of 8, have zero weight: every gate
+            # function maps (0, 0) to 0)
+            t["router_weight"], (_, self.shared_at, _) = pack_rows([t["router_weight"], gu[:f], gu[f:]])
+            if pad:
+                t["shared_down_weight"] = torch.nn.functional.pad(t["shared_down_weight"], (0, pad)).contiguous()
         elif self.shared_inner:
             # the shared feed-forward's gate is one more row of the router; rows up to a multiple of 8 are zero
             rows = [t["router_weight"], t.pop("shared_gate_weight")]
@@ -210,7 +214,7 @@ class MixtureOfExperts(Part):
 
     def _route(self, ctx, h):
         """Routing by the router: (weights, tiles, meta, row_token, place_of, weights by place or ``None``, the shared
-        feed-forward's gate logits or ``None``)."""
+        feed-forward's gate logits or ``None``, the whole of the router's product)."""
         n, E, top = ctx.n_tokens, self.num_experts, self.top
         ws, i32 = ctx.workspace, torch.int32
         ids = ws.get("moe_ids", (n * top,), i32)
@@ -235,7 +239,7 @@ class MixtureOfExperts(Part):
             K.moe_select(z, self.correction, counts=counts, **choice)
             K.moe_plan(ids, counts, fill, offsets, tiles, meta, row_token, place_of, n_tokens=n, n_experts=E, top=top,
                        weights=weights if self.weight_input else None, place_weight=by_place)
-        return weights, tiles, meta, row_token, place_of, by_place, full[:, E] if self.shared_inner and not self.gated else None
+        return weights, tiles, meta, row_token, place_of, by_place, full[:, E] if self.shared_inner and not self.gated else None, full
 
     def _experts(self, ctx, h, x, add: bool):
         """The experts' outputs, summed into ``x``, or (``x`` ``None``) left unsummed as a ``K.ExpertSum``."""
@@ -245,16 +249,14 @@ class MixtureOfExperts(Part):
         if self.routing == "table":
             weights, tiles, meta, row_token, place_of = self._table_route(ctx)
         else:
-            weights, tiles, meta, row_token, place_of, by_place, shared_gate = self._route(ctx, h)
+            weights, tiles, meta, row_token, place_of, by_place, shared_gate, full = self._route(ctx, h)
         if self.weight_input:
             weights = None
         if self.shared_inner:
             u = ws.get("moe_shared_inner", (n, self.shared_padded), ctx.act_dtype)
             if self.gated_shared:
-                gu = ws.get("moe_shared_gate_up", (n, 2 * self.shared_padded), ctx.act_dtype)
-                K.linear(h, self.shared_gate_up_weight, None, gu)
-                K.gated_act(gu, u, width=self.shared_padded, up_at=self.shared_padded, gate=self.gate, alpha=self.alpha,
-                            limit=self.limit)
+                K.gated_act(full[:, self.shared_at:], u, width=self.shared_padded, up_at=self.shared_padded, gate=self.gate,
+                            alpha=self.alpha, limit=self.limit)
             else:
                 K.linear(h, self.shared_up_weight, None, u, act=self.shared_act)
             shared = ws.get("moe_shared_out", (n, hid), torch.float32)
@@ -270,7 +272,8 @@ class MixtureOfExperts(Part):
         self._experts(ctx, h, x, add)
 
     def forward_deferred(self, ctx, h) -> "K.ExpertSum":
-        """Everything but the sum of a token's experts, for a consumer that forms it itself."""
+        """Everything but the sum of a token's experts, for a consumer that forms it itself (a block whose norm behind the
+        sublayer ``takes_expert_sum``)."""
         return self._experts(ctx, h, None, False)
 
 

@@ -286,14 +286,25 @@ class RMSNorm(Part):
         K.rmsnorm(x, self.weight, self.eps, out, rows)
         return out
 
+    def takes_expert_sum(self) -> bool:
+        """Whether ``add_to`` (factor 1, no copy) and ``add_then_norm`` take a ``K.ExpertSum`` in place of summed rows."""
+        return K.rmsnorm_add_experts_fits(self.hidden_size)
+
     def add_to(self, ctx, y, x, mult: float, copy=None) -> None:
+        if isinstance(y, K.ExpertSum):
+            if mult != 1.0 or copy is not None:
+                raise ValueError("rms_norm: a mixture of experts not yet summed is added with a factor of 1 and no copy")
+            K.rmsnorm_add_experts(y, self.weight, self.eps, x)
+            return
         K.rmsnorm_add(y, self.weight, self.eps, x, mult, copy)
 
     def add_then_norm(self, ctx, y, x, following: "RMSNorm", name: str = "normed"):
         """``x += norm(y)`` and, in the same pass, the new rows normalised by ``following`` (the norm
         ahead of the next sublayer) in the activation dtype."""
         out = ctx.workspace.get(name, tuple(x.shape), ctx.act_dtype)
-        if self.hidden_size > K.RMSNORM_ADD_NORM_MAX_WIDTH:
+        if isinstance(y, K.ExpertSum):
+            K.rmsnorm_add_experts(y, self.weight, self.eps, x, following.weight, following.eps, out)
+        elif self.hidden_size > K.RMSNORM_ADD_NORM_MAX_WIDTH:
             K.rmsnorm_add(y, self.weight, self.eps, x, 1.0, None)
             K.rmsnorm(x, following.weight, following.eps, out)
         else:
@@ -678,7 +689,8 @@ class PrePostNormBlock(Part):
     """Norms on both sides of every sublayer: ``x += norm_out(mixer(norm(x)))``, then (where the layer has
     a feed-forward) ``x += norm_out(feed_forward(norm(x)))``, four norms of their own.  A norm behind a
     sublayer and the norm ahead of the next one (the feed-forward's, or the first norm of the layer that
-    runs next) are one kernel: a layer launches two norm kernels, the model's first layer three."""
+    runs next) are one kernel: a layer launches two norm kernels, the model's first layer three.  A mixture of experts
+    leaves the sum over a token's experts to that kernel."""
 
     graph_safe = True
     launches_replayable = True
@@ -703,8 +715,12 @@ class PrePostNormBlock(Part):
             else:
                 last.add_to(ctx, y, x, 1.0)
                 h = layer.norm_feed_forward.forward(ctx, x)
-            layer.feed_forward.forward(ctx, h, y, add=False)
             last = layer.norm_feed_forward_out
+            deferred = getattr(layer.feed_forward, "forward_deferred", None)
+            if deferred is not None and getattr(last, "takes_expert_sum", None) is not None and last.takes_expert_sum():
+                y = deferred(ctx, h)
+            else:
+                layer.feed_forward.forward(ctx, h, y, add=False)
         # the layer's last addition to the stream, in one kernel with the first norm of the layer that runs next
         # where that layer is arranged the same way
         nxt = ctx.extras.get("next_layer")

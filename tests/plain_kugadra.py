@@ -19,7 +19,7 @@ import torch
 F64 = torch.float64
 
 # Where an engine that keeps activations in 16 bits rounds them (rows that matrix products read, cached latents, the
-# mixers' results ahead of their output products, inner rows of the feed-forwards): the identity, or a function that
+# linear attention's queries, keys and values, the mixers' results ahead of their output products, inner rows of the feed-forwards): the identity, or a function that
 # rounds, to see how far such rounding alone moves the logits of a sequence.
 _round = lambda t: t
 
@@ -55,8 +55,8 @@ def lightning(h: torch.Tensor, w: dict, p: str, m: dict, eps: float) -> torch.Te
     """silu on all three projections; the merged heads' norm is over all of their columns together; gate; output."""
     T, h = h.shape[0], _round(h)
     H, dk, dv = m["heads"], m["dim"], m["vdim"]
-    q, k = (silu(h @ w[p + n].T).view(T, H, dk) for n in ("q", "k"))
-    v = silu(h @ w[p + "v"].T).view(T, H, dv)
+    q, k = (_round(silu(h @ w[p + n].T)).view(T, H, dk) for n in ("q", "k"))
+    v = _round(silu(h @ w[p + "v"].T)).view(T, H, dv)
     o, _ = decayed_states(q, k, v, m["decay"])
     o = norm(o.reshape(T, H * dv), w[p + "norm"], eps) * torch.sigmoid(h @ w[p + "g"].T)
     return _round(o) @ w[p + "o"].T
