@@ -181,7 +181,13 @@ __global__ __launch_bounds__(256) void lightning_scan_kernel(const LightningPara
 
 // ---- the tensor cores -------------------------------------------------------------------------------------------
 
-constexpr int LG_N = 64, LG_LDV = LG_N + 8;  // value columns a block, row of a value or state tile in shared memory
+// A block has NG groups of four warps, each group 64 value columns: the queries and keys of a chunk are brought in once
+// for all of them.
+constexpr int LG_N = 64;
+template <int NG>
+struct LightningCols {
+  static constexpr int N = LG_N * NG, LD = N + 8;  // value columns a block, row of a value or state tile in shared memory
+};
 
 __device__ __forceinline__ void ldmatrix_x4_trans(uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3, const void* row) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
@@ -196,24 +202,40 @@ __device__ __forceinline__ uint32_t pack2(float lo, float hi) {
   const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
   return *reinterpret_cast<const uint32_t*>(&v);
 }
-// `rows` x `cols` elements f(row, column) of a float32 matrix into a bfloat16 tile of 64 (or `rows_pad`) rows, zeros outside.
-// VEC: columns in fours, 16-byte loads.
+// `rows` x `cols` elements of a float32 matrix, handed to put(row, column, values) for a tile of `rows_pad` x `cols_pad`, zeros
+// outside.  VEC: columns in fours, 16-byte loads.  A thread has eight pieces on their way before it uses the first.
 template <bool VEC, class Put>
 __device__ __forceinline__ void lightning_stage(const float* src, long ld, int rows, int cols, int rows_pad, int cols_pad, Put put) {
-  constexpr int W = VEC ? 4 : 1;
-  const int per_row = cols_pad / W;
-  for (int i = threadIdx.x; i < rows_pad * per_row; i += blockDim.x) {
-    const int r = i / per_row, c = (i - r * per_row) * W;
-    float x[W] = {};
-    if (r < rows && c < cols) {
-      if constexpr (VEC) {
-        const float4 f = *reinterpret_cast<const float4*>(src + (size_t)r * ld + c);
-        x[0] = f.x, x[1] = f.y, x[2] = f.z, x[3] = f.w;
-      } else {
-        x[0] = src[(size_t)r * ld + c];
-      }
+  constexpr int W = VEC ? 4 : 1, BATCH = 8;
+  const int per_row = cols_pad / W, dr = blockDim.x / per_row, dc = blockDim.x - dr * per_row;
+  int r0 = threadIdx.x / per_row, c0 = threadIdx.x - r0 * per_row;
+  auto advance = [&](int& r, int& c) {
+    r += dr;
+    c += dc;
+    if (c >= per_row) {
+      c -= per_row;
+      ++r;
     }
-    put(r, c, x);
+  };
+  while (r0 < rows_pad) {
+    float x[BATCH][W];
+    int r = r0, c = c0;
+#pragma unroll
+    for (int b = 0; b < BATCH; ++b) {
+      const bool in = r < rows && c * W < cols;
+      if constexpr (VEC) {
+        const float4 f = in ? *reinterpret_cast<const float4*>(src + (size_t)r * ld + c * W) : make_float4(0.f, 0.f, 0.f, 0.f);
+        x[b][0] = f.x, x[b][1] = f.y, x[b][2] = f.z, x[b][3] = f.w;
+      } else {
+        x[b][0] = in ? src[(size_t)r * ld + c] : 0.f;
+      }
+      advance(r, c);
+    }
+#pragma unroll
+    for (int b = 0; b < BATCH; ++b) {
+      if (r0 < rows_pad) put(r0, c0 * W, x[b]);
+      advance(r0, c0);
+    }
   }
 }
 template <int W>
@@ -234,13 +256,14 @@ __device__ __forceinline__ void store_split(__nv_bfloat16* hi, __nv_bfloat16* lo
   store_bf16(lo, rest);
 }
 
-// Grid (tiles, heads, groups of 64 value columns): U of the chunk, rows of 16 keys over the four warps in turn.
-template <bool VEC>
-__global__ __launch_bounds__(128) void lightning_chunk_mma_kernel(const LightningParams p, const int* __restrict__ tiles) {
+// Grid (tiles, heads, groups of 64 NG value columns): U of the chunk, rows of 16 keys over a group's four warps in turn.
+template <bool VEC, int NG>
+__global__ __launch_bounds__(128 * NG) void lightning_chunk_mma_kernel(const LightningParams p, const int* __restrict__ tiles) {
   extern __shared__ __align__(16) unsigned char lightning_smem[];
   __shared__ float pw_s[LG_C + 1];
   using bf16 = __nv_bfloat16;
-  const int h = blockIdx.y, n0 = blockIdx.z * LG_N;
+  constexpr int LDV = LightningCols<NG>::LD, COLS = LightningCols<NG>::N;
+  const int h = blockIdx.y, n0 = blockIdx.z * COLS;
   if (threadIdx.x <= LG_C) pw_s[threadIdx.x] = p.powers[h * (LG_C + 1) + threadIdx.x];
   pdl_begin();
   const LightningTile t = lightning_tile(p, tiles, blockIdx.x);
@@ -248,7 +271,7 @@ __global__ __launch_bounds__(128) void lightning_chunk_mma_kernel(const Lightnin
   const int dkp = (p.dk + 15) & ~15, LDK = dkp + 8;
   bf16* k_hi = reinterpret_cast<bf16*>(lightning_smem);  // [64][LDK]
   bf16* k_lo = k_hi + LG_C * LDK;
-  bf16* v_s = k_lo + LG_C * LDK;  // [64][LG_LDV]
+  bf16* v_s = k_lo + LG_C * LDK;  // [64][LDV]
   __syncthreads();
   const float* row = p.proj + (size_t)t.tok * p.ldp;
   lightning_stage<VEC>(row + p.off_k + h * p.dk, p.ldp, t.n, p.dk, LG_C, dkp, [&](int r, int c, auto& x) {
@@ -256,12 +279,13 @@ __global__ __launch_bounds__(128) void lightning_chunk_mma_kernel(const Lightnin
     for (auto& e : x) e = __bfloat162float(__float2bfloat16_rn(lightning_act_fast(e, p.act))) * w;  // the key as lightning_out_mma_kernel has it
     store_split(k_hi + r * LDK + c, k_lo + r * LDK + c, x);
   });
-  lightning_stage<VEC>(row + p.off_v + h * p.dv + n0, p.ldp, t.n, p.dv - n0, LG_C, LG_N, [&](int r, int c, auto& x) {
+  lightning_stage<VEC>(row + p.off_v + h * p.dv + n0, p.ldp, t.n, p.dv - n0, LG_C, COLS, [&](int r, int c, auto& x) {
     for (auto& e : x) e = lightning_act_fast(e, p.act);
-    store_bf16(v_s + r * LG_LDV + c, x);
+    store_bf16(v_s + r * LDV + c, x);
   });
   __syncthreads();
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, q2 = 2 * (lane & 3);
+  const int lane = threadIdx.x & 31, warp = (threadIdx.x >> 5) & 3, g = lane >> 2, q2 = 2 * (lane & 3);
+  const int v0 = (threadIdx.x >> 7) * LG_N;  // this group's first column in the tile
   float* u = p.chunks + ((size_t)blockIdx.x * p.n_heads + h) * p.dk * p.dv;
   for (int m0 = warp * 16; m0 < dkp; m0 += 64) {
     float acc[8][4] = {};
@@ -275,7 +299,7 @@ __global__ __launch_bounds__(128) void lightning_chunk_mma_kernel(const Lightnin
 #pragma unroll
       for (int nv = 0; nv < 8; nv += 2) {
         uint32_t b0, b1, b2, b3;
-        ldmatrix_x4_trans(b0, b1, b2, b3, v_s + (j0 + (lane & 15)) * LG_LDV + (nv + (lane >> 4)) * 8);
+        ldmatrix_x4_trans(b0, b1, b2, b3, v_s + (j0 + (lane & 15)) * LDV + v0 + (nv + (lane >> 4)) * 8);
         mma_kn(acc[nv], a_hi, b0, b1);
         mma_kn(acc[nv + 1], a_hi, b2, b3);
         mma_kn(acc[nv], a_lo, b0, b1);
@@ -286,7 +310,7 @@ __global__ __launch_bounds__(128) void lightning_chunk_mma_kernel(const Lightnin
     for (int nv = 0; nv < 8; ++nv)
 #pragma unroll
       for (int half = 0; half < 2; ++half) {
-        const int m = m0 + g + half * 8, n = n0 + nv * 8 + q2;
+        const int m = m0 + g + half * 8, n = n0 + v0 + nv * 8 + q2;
         if (m >= p.dk || n >= p.dv) continue;
         float* dst = u + (size_t)m * p.dv + n;
         if (VEC) {
@@ -299,22 +323,23 @@ __global__ __launch_bounds__(128) void lightning_chunk_mma_kernel(const Lightnin
   }
 }
 
-// Grid (tiles, heads, groups of 64 value columns): the chunk's outputs, 16 tokens a warp.
-template <bool VEC>
-__global__ __launch_bounds__(128) void lightning_out_mma_kernel(const LightningParams p, const int* __restrict__ tiles) {
+// Grid (tiles, heads, groups of 64 NG value columns): the chunk's outputs, 16 tokens and 64 columns a warp.
+template <bool VEC, int NG>
+__global__ __launch_bounds__(128 * NG) void lightning_out_mma_kernel(const LightningParams p, const int* __restrict__ tiles) {
   extern __shared__ __align__(16) unsigned char lightning_smem[];
   __shared__ float pw_s[LG_C + 1];
   using bf16 = __nv_bfloat16;
-  const int h = blockIdx.y, n0 = blockIdx.z * LG_N;
+  constexpr int LDV = LightningCols<NG>::LD, COLS = LightningCols<NG>::N;
+  const int h = blockIdx.y, n0 = blockIdx.z * COLS;
   if (threadIdx.x <= LG_C) pw_s[threadIdx.x] = p.powers[h * (LG_C + 1) + threadIdx.x];
   pdl_begin();
   const LightningTile t = lightning_tile(p, tiles, blockIdx.x);
   const int dkp = (p.dk + 15) & ~15, LDK = dkp + 8;
   bf16* q_s = reinterpret_cast<bf16*>(lightning_smem);  // [64][LDK]
   bf16* k_s = q_s + LG_C * LDK;                         // [64][LDK]
-  bf16* v_s = k_s + LG_C * LDK;                         // [64][LG_LDV]
-  bf16* st_hi = v_s + LG_C * LG_LDV;                    // [dkp][LG_LDV]
-  bf16* st_lo = st_hi + dkp * LG_LDV;
+  bf16* v_s = k_s + LG_C * LDK;                         // [64][LDV]
+  bf16* st_hi = v_s + LG_C * LDV;                    // [dkp][LDV]
+  bf16* st_lo = st_hi + dkp * LDV;
   const float* row = p.proj + (size_t)t.tok * p.ldp;
   const int live_rows = t.live ? t.n : 0;
   auto put_act = [&](bf16* dst, int ld) {
@@ -325,11 +350,12 @@ __global__ __launch_bounds__(128) void lightning_out_mma_kernel(const LightningP
   };
   lightning_stage<VEC>(row + p.off_q + h * p.dk, p.ldp, live_rows, p.dk, LG_C, dkp, put_act(q_s, LDK));
   lightning_stage<VEC>(row + p.off_k + h * p.dk, p.ldp, live_rows, p.dk, LG_C, dkp, put_act(k_s, LDK));
-  lightning_stage<VEC>(row + p.off_v + h * p.dv + n0, p.ldp, live_rows, p.dv - n0, LG_C, LG_N, put_act(v_s, LG_LDV));
-  lightning_stage<VEC>(p.chunks + ((size_t)blockIdx.x * p.n_heads + h) * p.dk * p.dv + n0, p.dv, t.live ? p.dk : 0, p.dv - n0, dkp, LG_N,
-                       [&](int r, int c, auto& x) { store_split(st_hi + r * LG_LDV + c, st_lo + r * LG_LDV + c, x); });
+  lightning_stage<VEC>(row + p.off_v + h * p.dv + n0, p.ldp, live_rows, p.dv - n0, LG_C, COLS, put_act(v_s, LDV));
+  lightning_stage<VEC>(p.chunks + ((size_t)blockIdx.x * p.n_heads + h) * p.dk * p.dv + n0, p.dv, t.live ? p.dk : 0, p.dv - n0, dkp, COLS,
+                       [&](int r, int c, auto& x) { store_split(st_hi + r * LDV + c, st_lo + r * LDV + c, x); });
   __syncthreads();
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, q2 = 2 * (lane & 3);
+  const int lane = threadIdx.x & 31, warp = (threadIdx.x >> 5) & 3, g = lane >> 2, q2 = 2 * (lane & 3);
+  const int v0 = (threadIdx.x >> 7) * LG_N;  // this group's first column in the tile
   if (warp * 16 >= t.n) return;
   const int row_a = warp * 16 + g, row_b = row_a + 8;  // tokens of the chunk
   const int key_tiles = 2 * (warp + 1);                // tiles of eight keys up to the warp's last token
@@ -349,7 +375,7 @@ __global__ __launch_bounds__(128) void lightning_out_mma_kernel(const LightningP
 #pragma unroll
     for (int nv = 0; nv < 8; nv += 2) {
       uint32_t b0, b1, b2, b3;
-      const int off = (c0 + (lane & 15)) * LG_LDV + (nv + (lane >> 4)) * 8;
+      const int off = (c0 + (lane & 15)) * LDV + v0 + (nv + (lane >> 4)) * 8;
       ldmatrix_x4_trans(b0, b1, b2, b3, st_hi + off);
       mma_kn(o[nv], a, b0, b1);
       mma_kn(o[nv + 1], a, b2, b3);
@@ -382,7 +408,7 @@ __global__ __launch_bounds__(128) void lightning_out_mma_kernel(const LightningP
 #pragma unroll
       for (int nv = 0; nv < 8; nv += 2) {
         uint32_t b0, b1, b2, b3;
-        ldmatrix_x4_trans(b0, b1, b2, b3, v_s + (nk * 8 + (lane & 15)) * LG_LDV + (nv + (lane >> 4)) * 8);
+        ldmatrix_x4_trans(b0, b1, b2, b3, v_s + (nk * 8 + (lane & 15)) * LDV + v0 + (nv + (lane >> 4)) * 8);
         mma_kn(o[nv], a_hi, b0, b1);
         mma_kn(o[nv + 1], a_hi, b2, b3);
         mma_kn(o[nv], a_lo, b0, b1);
@@ -394,7 +420,7 @@ __global__ __launch_bounds__(128) void lightning_out_mma_kernel(const LightningP
   for (int nv = 0; nv < 8; ++nv)
 #pragma unroll
     for (int half = 0; half < 2; ++half) {
-      const int i = half ? row_b : row_a, n = n0 + nv * 8 + q2;
+      const int i = half ? row_b : row_a, n = n0 + v0 + nv * 8 + q2;
       if (i >= t.n || n >= p.dv) continue;
       float* dst = p.out + (size_t)(t.tok + i) * p.n_heads * p.dv + (size_t)h * p.dv + n;
       if (VEC) {
@@ -567,13 +593,31 @@ static int lightning_sms() {
 
 template <class Kernel>
 static void lightning_mma_launch(Kernel kernel, bool& ready, dim3 grid, size_t smem, cudaStream_t stream, const LightningParams& p,
-                                 const int* tiles) {
+                                 const int* tiles, int groups) {
   if (!ready) {
     note_launch(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024));
     note_launch(cudaFuncSetAttribute(kernel, cudaFuncAttributePreferredSharedMemoryCarveout, (int)cudaSharedmemCarveoutMaxShared));
     ready = true;
   }
-  launch_pdl_split(false, kernel, grid, dim3(128), smem, stream, p, tiles);
+  launch_pdl_split(false, kernel, grid, dim3(128 * groups), smem, stream, p, tiles);
+}
+
+template <bool VEC, int NG, class Scan>
+static void lightning_mma_form(const LightningParams& p, const int* tiles, int n_tiles, cudaStream_t stream, Scan scan) {
+  static bool ready[2] = {false, false};
+  const int dkp = (p.dk + 15) & ~15, ldk = dkp + 8, ldv = LightningCols<NG>::LD;
+  const dim3 grid(n_tiles, p.n_heads, (p.dv + LightningCols<NG>::N - 1) / LightningCols<NG>::N);
+  lightning_mma_launch(lightning_chunk_mma_kernel<VEC, NG>, ready[0], grid, (size_t)(2 * LG_C * ldk + LG_C * ldv) * 2, stream, p, tiles, NG);
+  scan();
+  lightning_mma_launch(lightning_out_mma_kernel<VEC, NG>, ready[1], grid, (size_t)(2 * LG_C * ldk + (LG_C + 2 * dkp) * ldv) * 2, stream, p,
+                       tiles, NG);
+}
+template <class Scan>
+static void lightning_mma(bool vec, bool wide, const LightningParams& p, const int* tiles, int n_tiles, cudaStream_t stream, Scan scan) {
+  if (vec && wide) lightning_mma_form<true, 2>(p, tiles, n_tiles, stream, scan);
+  else if (vec) lightning_mma_form<true, 1>(p, tiles, n_tiles, stream, scan);
+  else if (wide) lightning_mma_form<false, 2>(p, tiles, n_tiles, stream, scan);
+  else lightning_mma_form<false, 1>(p, tiles, n_tiles, stream, scan);
 }
 
 }  // namespace rl
@@ -599,16 +643,11 @@ RL_EXPORT int rl_lightning(const float* proj, long ldp, int off_q, int off_k, in
     if (tensor_cores) {
       const bool vec = state4 && dk % 4 == 0 && ldp % 4 == 0 && off_q % 4 == 0 && off_k % 4 == 0 && off_v % 4 == 0 &&
                        (uintptr_t)proj % 16 == 0 && (uintptr_t)chunks % 16 == 0 && (uintptr_t)out % 16 == 0;
-      const int dkp = (dk + 15) & ~15, ldk = dkp + 8;
-      static bool ready[4] = {false, false, false, false};
-      const size_t s1 = (size_t)(2 * rl::LG_C * ldk + rl::LG_C * rl::LG_LDV) * 2;
-      const size_t s2 = (size_t)(2 * rl::LG_C * ldk + (rl::LG_C + 2 * dkp) * rl::LG_LDV) * 2;
-      rl::lightning_mma_launch(vec ? rl::lightning_chunk_mma_kernel<true> : rl::lightning_chunk_mma_kernel<false>, ready[vec], out_grid,
-                               s1, stream, p, tiles);
-      rl::launch_pdl(state4 ? rl::lightning_scan_kernel<4> : rl::lightning_scan_kernel<1>,
-                     dim3(n_tiles, n_heads, (dk * dv / (state4 ? 4 : 1) + 255) / 256), 256, 0, stream, p, tiles);
-      rl::lightning_mma_launch(vec ? rl::lightning_out_mma_kernel<true> : rl::lightning_out_mma_kernel<false>, ready[2 + vec], out_grid,
-                               s2, stream, p, tiles);
+      const bool wide = dv > 64 && dk <= 128;  // two groups of columns a block, where its shared memory has room for their states
+      rl::lightning_mma(vec, wide, p, tiles, n_tiles, stream, [&] {
+        rl::launch_pdl(state4 ? rl::lightning_scan_kernel<4> : rl::lightning_scan_kernel<1>,
+                       dim3(n_tiles, n_heads, (dk * dv / (state4 ? 4 : 1) + 255) / 256), 256, 0, stream, p, tiles);
+      });
     } else {
       rl::launch_pdl(rl::lightning_chunk_simt_kernel, dim3(n_tiles, n_heads, (dk + 63) / 64 * groups), 256, 0, stream, p, tiles);
       rl::launch_pdl(state4 ? rl::lightning_scan_kernel<4> : rl::lightning_scan_kernel<1>,

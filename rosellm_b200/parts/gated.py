@@ -265,7 +265,8 @@ class MixtureOfExperts(Part):
         eo = ws.get("moe_expert_out", (n * top, hid), torch.float32)
         K.moe_experts(h, self.gate_up_weight, self.down_weight, tiles, meta, row_token, place_of, weights, act, eo, x,
                       n_experts=E, top=top, ff=f, gate=self.gate, alpha=self.alpha, limit=self.limit, add=add,
-                      place_weight=by_place, shared=shared if x is not None else None, shared_gate=shared_gate)
+                      place_weight=by_place, shared=shared if x is not None else None,
+                      shared_gate=shared_gate if x is not None else None)
         return None if x is not None else K.ExpertSum(eo, weights, place_of, top, shared, shared_gate)
 
     def forward(self, ctx, h, x, add: bool = True) -> None:
