@@ -129,19 +129,29 @@ __global__ __launch_bounds__(256) void lightning_out_simt_kernel(const Lightning
 
 // ---- the states between the chunks ------------------------------------------------------------------------------
 
-// Grid (tiles, heads, pieces of a head's state): the blocks of a portion's first tile walk its tiles, a thread VEC
-// elements of the state, eight chunks' worth fetched at a time.
+// Grid (requests, heads, pieces of a head's state): a block walks its request's tiles, a thread VEC elements of the state,
+// eight chunks' worth fetched at a time.  The tiles lie request by request, so a request's first one is the number of
+// tiles of the requests before it (one token: none).
 template <int VEC>
-__global__ __launch_bounds__(256) void lightning_scan_kernel(const LightningParams p, const int* __restrict__ tiles) {
+__global__ __launch_bounds__(256) void lightning_scan_kernel(const LightningParams p) {
+  __shared__ int first_s;
   pdl_begin();
-  const int i0 = blockIdx.x;
-  if (tiles[2 * i0 + 1] != 0) return;
-  const int req = tiles[2 * i0], slot = p.slots[req];
-  if (slot < 0) return;
-  const int h = blockIdx.y, size = p.dk * p.dv;
+  const int req = blockIdx.x, slot = p.slots[req];
+  const int n_tok = p.q_start[req + 1] - p.q_start[req];
+  if (slot < 0 || n_tok < 2) return;
+  if (threadIdx.x == 0) first_s = 0;
+  __syncthreads();
+  int before = 0;
+  for (int r = threadIdx.x; r < req; r += blockDim.x) {
+    const int n = p.q_start[r + 1] - p.q_start[r];
+    before += n > 1 ? (n + LG_C - 1) / LG_C : 0;
+  }
+  if (before) atomicAdd(&first_s, before);
+  __syncthreads();
+  const int i0 = first_s, h = blockIdx.y, size = p.dk * p.dv;
   const int at = (blockIdx.z * blockDim.x + threadIdx.x) * VEC;
   if (at >= size) return;
-  const int n_tok = p.q_start[req + 1] - p.q_start[req], n_chunks = (n_tok + LG_C - 1) / LG_C;
+  const int n_chunks = (n_tok + LG_C - 1) / LG_C;
   const float* pw = p.powers + h * (LG_C + 1);
   const float d_full = pw[LG_C], d_last = pw[n_tok - (n_chunks - 1) * LG_C];
   float* st = p.state + (size_t)slot * p.state_stride + (size_t)h * size + at;
@@ -625,13 +635,13 @@ static void lightning_mma(bool vec, bool wide, const LightningParams& p, const i
 // One step for every request of the step.  proj float32 [tokens, ldp] with the queries, keys (heads * dk columns each)
 // and values (heads * dv) from the given columns on; act: 1 for silu on all three, 0 for none; powers float32 [heads,
 // 65], powers[h][n] = d_h^n; state float32, state_stride floats a slot; tiles [n_tiles][2]: (request, first token) of the
-// 64-token tiles of portions, a portion's tiles one after the other; decode_reqs: requests with one token; chunks: float32
+// 64-token tiles of all requests with more than one token, in the requests' and the tokens' order; decode_reqs: requests with one token; chunks: float32
 // scratch [n_tiles, heads, dk, dv]; out float32 [tokens, heads * dv].  tensor_cores: portions on the bfloat16 operands.
 RL_EXPORT int rl_lightning(const float* proj, long ldp, int off_q, int off_k, int off_v, int act, const float* powers,
-                           float* state, long state_stride, const int* q_start, const int* slots, const int* tiles, int n_tiles,
+                           float* state, long state_stride, const int* q_start, const int* slots, int n_reqs, const int* tiles, int n_tiles,
                            const int* decode_reqs, int n_decode, float* chunks, float* out, int n_heads, int dk, int dv,
                            int tensor_cores, cudaStream_t stream) {
-  if (n_heads <= 0 || n_heads > 65535 || dk <= 0 || dk > 256 || dv <= 0 || dv > 256 || n_tiles < 0 || n_decode < 0 ||
+  if (n_heads <= 0 || n_heads > 65535 || dk <= 0 || dk > 256 || dv <= 0 || dv > 256 || n_tiles < 0 || n_decode < 0 || n_reqs < 0 ||
       state_stride < (long)n_heads * dk * dv || (n_tiles > 0 && chunks == nullptr))
     return -2;
   const rl::LightningParams p{proj, ldp, off_q, off_k, off_v, powers, state, state_stride, chunks, out, q_start, slots,
@@ -640,18 +650,18 @@ RL_EXPORT int rl_lightning(const float* proj, long ldp, int off_q, int off_k, in
   if (n_tiles > 0) {
     const int groups = (dv + 63) / 64;
     const dim3 out_grid(n_tiles, n_heads, groups);
+    auto scan = [&] {
+      rl::launch_pdl(state4 ? rl::lightning_scan_kernel<4> : rl::lightning_scan_kernel<1>,
+                     dim3(n_reqs, n_heads, (dk * dv / (state4 ? 4 : 1) + 255) / 256), 256, 0, stream, p);
+    };
     if (tensor_cores) {
       const bool vec = state4 && dk % 4 == 0 && ldp % 4 == 0 && off_q % 4 == 0 && off_k % 4 == 0 && off_v % 4 == 0 &&
                        (uintptr_t)proj % 16 == 0 && (uintptr_t)chunks % 16 == 0 && (uintptr_t)out % 16 == 0;
       const bool wide = dv > 64 && dk <= 128;  // two groups of columns a block, where its shared memory has room for their states
-      rl::lightning_mma(vec, wide, p, tiles, n_tiles, stream, [&] {
-        rl::launch_pdl(state4 ? rl::lightning_scan_kernel<4> : rl::lightning_scan_kernel<1>,
-                       dim3(n_tiles, n_heads, (dk * dv / (state4 ? 4 : 1) + 255) / 256), 256, 0, stream, p, tiles);
-      });
+      rl::lightning_mma(vec, wide, p, tiles, n_tiles, stream, scan);
     } else {
       rl::launch_pdl(rl::lightning_chunk_simt_kernel, dim3(n_tiles, n_heads, (dk + 63) / 64 * groups), 256, 0, stream, p, tiles);
-      rl::launch_pdl(state4 ? rl::lightning_scan_kernel<4> : rl::lightning_scan_kernel<1>,
-                     dim3(n_tiles, n_heads, (dk * dv / (state4 ? 4 : 1) + 255) / 256), 256, 0, stream, p, tiles);
+      scan();
       rl::launch_pdl(rl::lightning_out_simt_kernel, out_grid, 256, 0, stream, p, tiles);
     }
   }

@@ -176,7 +176,7 @@ def _lib() -> ctypes.CDLL:
         lib.rl_recurrence.argtypes = [I, I, P, L, I, I, I, I, I, I, P, P, P, I, P, P, P, L, P, P, P, P, I, I, I, I, I, F, F, F,
                                       L, I, F, F, F, F, P, P]
         lib.rl_recurrence_record.argtypes = [I, I, I, P, P, P]
-        lib.rl_lightning.argtypes = [P, L, I, I, I, I, P, P, L, P, P, P, I, P, I, P, P, I, I, I, I, P]
+        lib.rl_lightning.argtypes = [P, L, I, I, I, I, P, P, L, P, P, I, P, I, P, I, P, P, I, I, I, I, P]
         lib.rl_rmsnorm_gate.argtypes = [I, P, L, P, L, P, P, L, I, I, F, P]
         lib.rl_soft_cap.argtypes = [P, L, F, P]
         lib.rl_bias_attention_shape.argtypes = [I, I, P, P]
@@ -1582,8 +1582,8 @@ def lightning(proj, offsets: dict, powers, state, q_start, slots, chunks, out, *
     """One step of linear attention with a fixed decay a head (csrc/lightning.cu) for every request of the step.
     ``proj`` float32 [tokens, columns], ``offsets`` the first column of ``q``, ``k`` and ``v``; ``powers`` float32
     [heads, 65]: the decays' powers 0 to 64; ``state`` float32 [slots, heads, dk, dv]; ``chunks`` float32 scratch of
-    n_tiles * heads * dk * dv floats (``None`` without portions); ``out`` float32 [tokens, heads * dv]; ``tiles``: the
-    step's 64-token tiles.  ``silu``: applied to the three projections.  ``tensor_cores``: portions of prompts with
+    n_tiles * heads * dk * dv floats (``None`` without portions); ``out`` float32 [tokens, heads * dv]; ``slots``
+    [requests]; ``tiles``: the step's 64-token tiles (of every request with more than one token).  ``silu``: applied to the three projections.  ``tensor_cores``: portions of prompts with
     queries, keys and values as bfloat16 operands."""
     for t, name in ((powers, "powers"), (state, "state"), (out, "out")):
         _need(t, name, torch.float32)
@@ -1600,7 +1600,7 @@ def lightning(proj, offsets: dict, powers, state, q_start, slots, chunks, out, *
         if chunks.numel() < n_tiles * n_heads * dk * dv:
             raise KernelError("lightning: scratch too small")
     rc = _lib().rl_lightning(_ptr(proj), proj.stride(0), *off, int(silu), _ptr(powers), _ptr(state), state.stride(0),
-                             _ptr(q_start), _ptr(slots), _ptr(tiles), n_tiles, _ptr(decode_reqs), n_decode, _ptr(chunks),
+                             _ptr(q_start), _ptr(slots), slots.numel(), _ptr(tiles), n_tiles, _ptr(decode_reqs), n_decode, _ptr(chunks),
                              _ptr(out), n_heads, dk, dv, int(tensor_cores), _stream())
     if rc == -2:
         raise KernelError(f"lightning: sizes not taken (key size {dk}, value size {dv}: up to 256 each)")
